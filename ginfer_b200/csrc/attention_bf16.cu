@@ -47,8 +47,9 @@ template <int MAXC>
 __device__ __forceinline__ void cluster_merge(float* cpart, float* cpart_m, float* cpart_l,
                                               float* cw, float* cinv, bf16* __restrict__ out,
                                               int nrows, int splits, int split, int row, int nh,
-                                              int h0, bool active = true, float* part_o = nullptr,
-                                              float* part_ml = nullptr, int parts = 1) {
+                                              int h0, float sink, bool active = true,
+                                              float* part_o = nullptr, float* part_ml = nullptr,
+                                              int parts = 1) {
   // Loads from the peers are issued eight at a time without branches (the peer index is
   // clamped, a clamped load's weight is zero); the additions stay in split order.
   // (`active` false: a thread beyond the NTHREADS that work here; it only joins the barrier)
@@ -72,7 +73,7 @@ __device__ __forceinline__ void cluster_merge(float* cpart, float* cpart_m, floa
       cw[r * 16 + p] = wgt;
       lsum += wgt * lp[p];
     }
-    cinv[r] = lsum > 0.f ? 1.f / lsum : 0.f;
+    cinv[r] = lsum > 0.f ? 1.f / (lsum + sink_share(sink, mm)) : 0.f;
     // part_o / part_ml: this cluster holds only a part of the request's keys; it leaves its
     // unnormalised result with the maximum and the sum for the kernel that merges the parts
     // (both pointers stand at this cluster's part of its first head; a head has `parts` parts)
@@ -338,7 +339,8 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16* __r
     }
     const int head = h0 + r;
     if (splits == 1) {
-      out[((size_t)row * nh + head) * HD + d] = __float2bfloat16_rn(lsum > 0.f ? acc / lsum : 0.f);
+      out[((size_t)row * nh + head) * HD + d] =
+          __float2bfloat16_rn(lsum > 0.f ? acc / (lsum + sink_share(shape.sink, mm)) : 0.f);
     } else if (fused_merge == 2) {
       cpart[i] = acc;                                   // this CTA's partial stays in shared memory
       if (d == 0) {
@@ -362,9 +364,11 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16* __r
     float* cw = cpart_l + 16;                           // [16 rows][16 splits] weights
     float* cinv = cw + 256;                             // [16]
     if (splits <= 8)
-      cluster_merge<8>(cpart, cpart_m, cpart_l, cw, cinv, out, nrows, splits, split, row, nh, h0);
+      cluster_merge<8>(cpart, cpart_m, cpart_l, cw, cinv, out, nrows, splits, split, row, nh, h0,
+                       shape.sink);
     else
-      cluster_merge<16>(cpart, cpart_m, cpart_l, cw, cinv, out, nrows, splits, split, row, nh, h0);
+      cluster_merge<16>(cpart, cpart_m, cpart_l, cw, cinv, out, nrows, splits, split, row, nh, h0,
+                        shape.sink);
     cluster_sync_all();                                 // nobody leaves while a peer reads it
     return;
   }
@@ -405,7 +409,7 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16* __r
       w[r * used + s2] = wgt;
       lsum += wgt * __ldcg(pml + (base + s2) * 2 + 1);
     }
-    linv[r] = lsum > 0.f ? 1.f / lsum : 0.f;
+    linv[r] = lsum > 0.f ? 1.f / (lsum + sink_share(shape.sink, mm)) : 0.f;
   }
   __syncthreads();
   for (int i = threadIdx.x; i < nrows * HD; i += NTHREADS) {
@@ -468,7 +472,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap,
                        bf16* __restrict__ out, int nh, int nkv, int page_size, int window,
                        float scale_log2, int splits, int oob_row, int tbl_cap, int nst,
                        int* err, const RopeArgs rope, int parts, float* __restrict__ po,
-                       float* __restrict__ pml) {
+                       float* __restrict__ pml, float sink) {
   // No static shared memory in this kernel: the dynamic part then starts at the aligned base,
   // which the swizzled tiles need (checked below: a misaligned base ends the CTA with code 5).
   extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -790,7 +794,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap,
       }
     } else if (splits == 1) {
       out[((size_t)row * nh + h0 + r) * HD + d] =
-          __float2bfloat16_rn(lsum > 0.f ? acc / lsum : 0.f);
+          __float2bfloat16_rn(lsum > 0.f ? acc / (lsum + sink_share(sink, mm)) : 0.f);
     } else {
       cpart[i] = acc;
       if (d == 0) {
@@ -805,10 +809,10 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap,
     cluster_sync_all();          // also orders the weights above before they are overwritten
     if (splits <= 8)
       cluster_merge<8>(cpart, cpart_m, cpart_l, cw, cinv, out, nrows, splits, split, row, nh, h0,
-                       consumer, part_o, part_ml, parts);
+                       sink, consumer, part_o, part_ml, parts);
     else
       cluster_merge<16>(cpart, cpart_m, cpart_l, cw, cinv, out, nrows, splits, split, row, nh, h0,
-                        consumer, part_o, part_ml, parts);
+                        sink, consumer, part_o, part_ml, parts);
     cluster_sync_all();          // nobody leaves while a peer reads it
   }
 }
@@ -818,7 +822,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap,
 __global__ void attn_decode_merge_kernel(const float* __restrict__ po,
                                          const float* __restrict__ pml,
                                          const int* __restrict__ cu_seqlens_q,
-                                         bf16* __restrict__ out, int nh, int splits) {
+                                         bf16* __restrict__ out, int nh, int splits,
+                                         float sink) {
   const int head = blockIdx.x, b = blockIdx.y, d = threadIdx.x;
   pdl_trigger();
   pdl_wait();
@@ -836,7 +841,8 @@ __global__ void attn_decode_merge_kernel(const float* __restrict__ po,
     lsum += wgt * pml[(base + s) * 2 + 1];
   }
   const int row = cu_seqlens_q ? cu_seqlens_q[b] : b;
-  out[((size_t)row * nh + head) * HD + d] = __float2bfloat16_rn(lsum > 0.f ? acc / lsum : 0.f);
+  out[((size_t)row * nh + head) * HD + d] =
+      __float2bfloat16_rn(lsum > 0.f ? acc / (lsum + sink_share(sink, mm)) : 0.f);
 }
 
 // ================================================================================== prefill
@@ -1025,7 +1031,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16* __
       li += __shfl_xor_sync(0xffffffffu, li, 2);
       const int r = warp * WROWS + mt * 16 + g + 8 * i;
       if (r >= rows) continue;
-      const float inv = li > 0.f ? 1.f / li : 0.f;
+      const float inv = li > 0.f ? 1.f / (li + sink_share(shape.sink, m[mt][i])) : 0.f;
       bf16* orow = out + ((size_t)(q_begin + r0 + r) * nh + head) * HD;
 #pragma unroll
       for (int n = 0; n < HD / 8; ++n) {
@@ -1058,7 +1064,7 @@ static int attn_decode_impl(const void* q, int q_row_stride, const void* kpages,
                             const int* cu_seqlens_q, const int* positions, void* out,
                             void* scratch, int B, int nh, int nkv, int page_size, int window,
                             float scale, int splits, const RopeArgs& rope, void* stream,
-                            const ScoreShape shape = ScoreShape{0.f, nullptr}) {
+                            const ScoreShape shape = ScoreShape{0.f, nullptr, kNoSink}) {
   if (B <= 0) return 0;
   if (nkv <= 0 || nh <= 0 || nh % nkv || splits < 1) return -3;
   auto st = (cudaStream_t)stream;
@@ -1114,21 +1120,21 @@ static int attn_decode_impl(const void* q, int q_row_stride, const void* kpages,
                          shape);
   if (rc || splits == 1 || fused) return rc;
   return launch_kernel(attn_decode_merge_kernel, dim3(nh, B), dim3(HD), 0, st, (const float*)po,
-                       (const float*)pml, cu_seqlens_q, (bf16*)out, nh, splits);
+                       (const float*)pml, cu_seqlens_q, (bf16*)out, nh, splits, shape.sink);
 }
 
 // The TMA kernel where it serves the case: head sizes that are a multiple of 64, page sizes that
 // are a multiple of 8 and divide (or are a multiple of) the 64-key tile, 1 split or a cluster of
 // 2, 4, 8 or 16.  -6: not served (the caller takes gf_attn_decode / gf_attn_decode_rope).
 // `stages`: depth of the ring of tiles (2 .. 6, cut to what shared memory holds; 3 lets two CTAs
-// share an SM).  `err` receives 4 or 6 if a wait for a tile or for a free stage ran out.
+// share an SM).  `sink`: the sink's score, -inf for none.  `err` receives 4 or 6 if a wait for a tile or for a free stage ran out.
 GF_EXPORT int gf_attn_decode_tma(const void* q, int q_row_stride, void* kpages, void* vpages,
                                  int num_pages, const int* block_table, int table_stride,
                                  const int* cu_seqlens_q, const int* positions, void* out, int B,
                                  int nh, int nkv, int page_size, int window, float scale,
                                  int splits, int stages, const float* rope_table, int rot,
                                  int fused, int write_kv, int* err, void* stream, int parts,
-                                 void* scratch) {
+                                 void* scratch, float sink) {
 #if GF_HEAD_DIM % 64 == 0
   if (B <= 0) return 0;
   if (nh % nkv || splits < 1 || parts < 1 || (parts > 1 && !scratch)) return -3;
@@ -1177,10 +1183,10 @@ GF_EXPORT int gf_attn_decode_tma(const void* q, int q_row_stride, void* kpages, 
                                       (bf16*)kpages, (bf16*)vpages, block_table, table_stride,
                                       cu_seqlens_q, positions, (bf16*)out, nh, nkv, page_size,
                                       window, scale * LOG2E, splits, (int)slots, tbl_cap, nst, err,
-                                      rope, parts, po, pml);
+                                      rope, parts, po, pml, sink);
   if (rc || parts == 1) return rc;
   return launch_kernel(attn_decode_merge_kernel, dim3(nh, B), dim3(HD), 0, st, (const float*)po,
-                       (const float*)pml, cu_seqlens_q, (bf16*)out, nh, parts);
+                       (const float*)pml, cu_seqlens_q, (bf16*)out, nh, parts, sink);
 #else
   return -6;
 #endif
@@ -1212,18 +1218,19 @@ GF_EXPORT int gf_attn_decode_rope(const void* q, int q_row_stride, void* kpages,
 }
 
 // gf_attn_decode with shaped scores: `softcap` > 0 caps them (cap * tanh(score / cap)), `slopes`
-// (fp32 [nh] or null) takes slope * (p - c) off the score of the key at c.
+// (fp32 [nh] or null) takes slope * (p - c) off the score of the key at c, `sink` (-inf: none) is
+// the score of a sink.
 GF_EXPORT int gf_attn_decode_shaped(const void* q, int q_row_stride, const void* kpages,
                                     const void* vpages, const int* block_table, int table_stride,
                                     const int* cu_seqlens_q, const int* positions, void* out,
                                     void* scratch, int B, int nh, int nkv, int page_size,
                                     int window, float scale, int splits, float softcap,
-                                    const float* slopes, void* stream) {
+                                    const float* slopes, float sink, void* stream) {
   if (softcap < 0.f) return -3;
   return attn_decode_impl(q, q_row_stride, kpages, vpages, block_table, table_stride,
                           cu_seqlens_q, positions, out, scratch, B, nh, nkv, page_size, window,
                           scale, splits, RopeArgs{nullptr, 0, 0, 0}, stream,
-                          ScoreShape{softcap, slopes});
+                          ScoreShape{softcap, slopes, sink});
 }
 
 static int attn_prefill_impl(const void* q, int q_row_stride, const void* kpages,
@@ -1258,7 +1265,7 @@ GF_EXPORT int gf_attn_prefill(const void* q, int q_row_stride, const void* kpage
                               float scale, void* stream) {
   return attn_prefill_impl(q, q_row_stride, kpages, vpages, block_table, table_stride,
                            cu_seqlens_q, kv_lens, out, B, max_q_len, nh, nkv, page_size, window,
-                           scale, stream, ScoreShape{0.f, nullptr});
+                           scale, stream, ScoreShape{0.f, nullptr, kNoSink});
 }
 
 // The same with shaped scores (see gf_attn_decode_shaped).
@@ -1267,11 +1274,11 @@ GF_EXPORT int gf_attn_prefill_shaped(const void* q, int q_row_stride, const void
                                      const int* cu_seqlens_q, const int* kv_lens, void* out,
                                      int B, int max_q_len, int nh, int nkv, int page_size,
                                      int window, float scale, float softcap, const float* slopes,
-                                     void* stream) {
+                                     float sink, void* stream) {
   if (softcap < 0.f) return -3;
   return attn_prefill_impl(q, q_row_stride, kpages, vpages, block_table, table_stride,
                            cu_seqlens_q, kv_lens, out, B, max_q_len, nh, nkv, page_size, window,
-                           scale, stream, ScoreShape{softcap, slopes});
+                           scale, stream, ScoreShape{softcap, slopes, sink});
 }
 
 // ----------------------------------------------------------------------------- no allocation

@@ -20,6 +20,11 @@ __device__ __forceinline__ uint32_t smem_u32(const void* p) {
   return (uint32_t)__cvta_generic_to_shared(p);
 }
 
+// xIELU: a z^2 + z/2 above zero, b (e^z - 1 - z) + z/2 below.
+__device__ __forceinline__ float xielu(float z, float a, float b) {
+  return (z > 0.f ? a * z * z : b * (expm1f(z) - z)) + 0.5f * z;
+}
+
 template <typename T> __device__ __forceinline__ float to_f32(T v);
 template <> __device__ __forceinline__ float to_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ float to_f32<__nv_bfloat16>(__nv_bfloat16 v) {
@@ -99,13 +104,22 @@ __host__ __device__ __forceinline__ int first_visible_key(int p, int span) {
 
 // Shaped attention scores.  With a cap, score <- cap * tanh(score / cap) after the scale; with
 // slopes (one a head), slope * (p - c) is then taken off the score of the key at c for the query at
-// p.  32-bit arithmetic in every kernel that takes it.
+// p.  A sink adds exp(sink) to the softmax's denominator: a key with this score and no value.
+// 32-bit arithmetic in every kernel that takes it.
 struct ScoreShape {
   float cap;              // 0: no cap
   const float* slopes;    // [heads], or null: no distance bias
+  float sink;             // the sink's score; kNoSink: none
 };
+constexpr float kNoSink = -__builtin_inff();
+// Whether single scores change (the sink only enters a row's sum, at its end).
 __host__ __device__ __forceinline__ bool shaped(const ScoreShape& sh) {
   return sh.cap > 0.f || sh.slopes != nullptr;
+}
+// What a sink adds to a row's sum of 2^(score - m) when everything is in log2 units; nothing for
+// kNoSink.  m is the row's reference maximum (finite: a query sees itself).
+__device__ __forceinline__ float sink_share(float sink, float m_log2) {
+  return exp2f(fmaf(sink, 1.4426950408889634f, -m_log2));
 }
 
 // ---- programmatic dependent launch -------------------------------------------------------------

@@ -1,4 +1,5 @@
-// Gated delta rule with one decay per head and key channel, over packed tokens of several requests.
+// Gated delta rule with one decay per head and key channel, or one per head, over packed tokens of
+// several requests.
 // A request's state lives in a slot: S [heads, D, Vd] in fp32 and the last (taps - 1) inputs of the
 // short convolutions, fp32 as well.
 //
@@ -7,6 +8,8 @@
 //                            the tap reaches) + SiLU on the q | k | v channels; q and k made unit
 //                            vectors per head (q also times D^-1/2); decay g = exp(-exp(A_log_h) *
 //                            softplus(a + dt_bias)); beta = sigmoid(b).  Everything leaves in fp32.
+//   delta_prepare_heads_kernel  the same with one decay a head, four channels a lane, a warp walking
+//                            over a run of tokens with the convolution's inputs in registers.
 //   delta_conv_state_kernel  a thread a (request, channel): the slot's last inputs after the step.
 //   delta_recurrence_kernel  per (request, head): S <- g * S (rows); u = beta (v - S^T k);
 //                            S <- S + k u^T; o = S^T q, token after token.  The columns of S are
@@ -26,9 +29,11 @@ struct DeltaDims {
   int channels;          // 2 G D + H Vd: the convolved columns q | k | v of a projection row
   int state_stride;      // floats a slot
   int conv_off;          // where the convolution inputs start in a slot
+  int a_ld;              // one decay a head: floats between two tokens of its pre-activations
 };
 
-// A warp a (token, unit): units 0 .. G-1 are q heads, G .. 2G-1 k heads, then H v heads, then H
+// ONE_DECAY: `a` holds a pre-activation a head (rows of a_ld floats), and one unit makes all heads'
+// decays.  A warp a (token, unit): units 0 .. G-1 are q heads, G .. 2G-1 k heads, then H v heads, then H
 // decay rows, then one unit for the betas.  No warp waits for another.
 template <typename T>
 __device__ __forceinline__ float conv_silu_at(const T* __restrict__ proj, int ld, int r, int i,
@@ -48,7 +53,7 @@ __device__ __forceinline__ float conv_silu_at(const T* __restrict__ proj, int ld
 constexpr int kPrepareWarps = 8;
 constexpr int kPrepareMaxPerLane = 8;              // head sizes up to 256
 
-template <typename T>
+template <typename T, bool ONE_DECAY>
 __global__ void delta_prepare_kernel(const T* __restrict__ proj, int ld, int b_off,
                                      const float* __restrict__ a, const float* __restrict__ conv_w,
                                      const float* __restrict__ dt_bias,
@@ -65,7 +70,7 @@ __global__ void delta_prepare_kernel(const T* __restrict__ proj, int ld, int b_o
   pdl_trigger();
   pdl_wait();
   const int G = dm.G, H = dm.H, D = dm.D, Vd = dm.Vd;
-  if (unit >= 2 * G + 2 * H + 1) return;
+  if (unit >= 2 * G + H + (ONE_DECAY ? 0 : H) + 1) return;
   const int b = seq_of_token[r];
   const int i = r - cu_seqlens[b];                // place in this step's portion
   const float* cs = state + (size_t)slot_ids[b] * dm.state_stride + dm.conv_off;
@@ -94,7 +99,7 @@ __global__ void delta_prepare_kernel(const T* __restrict__ proj, int ld, int b_o
     for (int j = lane; j < Vd; j += 32)
       v[((size_t)r * H + h) * Vd + j] =
           conv_silu_at(proj, ld, r, i, cs, conv_w, taps, CH, 2 * GD + h * Vd + j);
-  } else if (unit < 2 * G + 2 * H) {              // a head's decays
+  } else if (!ONE_DECAY && unit < 2 * G + 2 * H) {              // a head's decays
     const int h = unit - 2 * G - H;
     const float rate = expf(A_log[h]);
     for (int d = lane; d < D; d += 32) {
@@ -104,6 +109,128 @@ __global__ void delta_prepare_kernel(const T* __restrict__ proj, int ld, int b_o
   } else {
     for (int h = lane; h < H; h += 32)
       beta[(size_t)r * H + h] = sigmoid_f(to_f32(proj[(size_t)r * ld + b_off + h]));
+    if (ONE_DECAY)
+      for (int h = lane; h < H; h += 32)
+        g[(size_t)r * H + h] =
+            expf(-expf(A_log[h]) * softplus_f(a[(size_t)r * dm.a_ld + h] + dt_bias[h]));
+  }
+}
+
+// One decay a head, the projection's row in fp32 (q | k | v first, decay and beta columns at a_off
+// and b_off).  Units: G q heads, G k heads, H v heads, one for decays and betas.  A warp takes a unit
+// and `run` consecutive tokens; lanes own four channels (NQ times); the last TAPS - 1 inputs stay in
+// registers from token to token and come from the slot at a portion's start.  update_state (every
+// portion of the step is one token): the same lanes bring the slot's inputs up to date.
+// D, Vd, ld and the offsets are multiples of 4.
+template <int TAPS, int NQ>
+__global__ void __launch_bounds__(128)
+delta_prepare_heads_kernel(const float* __restrict__ proj, int ld, int a_off, int b_off,
+                           const float* __restrict__ conv_w, const float* __restrict__ dt_bias,
+                           const float* __restrict__ A_log, float* __restrict__ state,
+                           const int* __restrict__ seq_of_token,
+                           const int* __restrict__ cu_seqlens, const int* __restrict__ slot_ids,
+                           DeltaDims dm, int T, int run, int update_state, float* __restrict__ qn,
+                           float* __restrict__ kn, float* __restrict__ v, float* __restrict__ g,
+                           float* __restrict__ beta) {
+  constexpr int KEEP = TAPS - 1;
+  const int lane = threadIdx.x & 31;
+  const int G = dm.G, H = dm.H, D = dm.D, Vd = dm.Vd, GD = G * D;
+  const int unit = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int r0 = blockIdx.x * run, r1 = min(r0 + run, T);
+  const bool convolves = unit < 2 * G + H;
+  const int size = unit < 2 * G ? D : Vd;
+  const int ch0 = unit < 2 * G ? unit * D : 2 * GD + (unit - 2 * G) * Vd;
+  float w[NQ][4][TAPS];
+  if (convolves) {                                  // weights: before the wait
+#pragma unroll
+    for (int u = 0; u < NQ; ++u)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int d = 4 * (lane + 32 * u) + i;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[u][i][j] = d < size ? conv_w[(size_t)(ch0 + d) * TAPS + j] : 0.f;
+      }
+  }
+  // few tokens: the recurrence may start early.  In a prompt its long-lived blocks would land several
+  // to an SM on the first SMs that drain.
+  if (run == 1) pdl_trigger();
+  pdl_wait();
+  if (unit > 2 * G + H) return;
+  if (!convolves) {
+    for (int e = lane; e < (r1 - r0) * H; e += 32) {
+      const int r = r0 + e / H, h = e % H;
+      const float* row = proj + (size_t)r * ld;
+      beta[(size_t)r * H + h] = sigmoid_f(row[b_off + h]);
+      g[(size_t)r * H + h] = expf(-expf(A_log[h]) * softplus_f(row[a_off + h] + dt_bias[h]));
+    }
+    return;
+  }
+  float past[NQ][4][KEEP > 0 ? KEEP : 1];           // inputs of the tokens before, oldest first
+  for (int r = r0; r < r1; ++r) {
+    const int b = seq_of_token[r], start = cu_seqlens[b];
+    float* cs = state + (size_t)slot_ids[b] * dm.state_stride + dm.conv_off;
+    if (r == r0 || r == start) {
+#pragma unroll
+      for (int m = 0; m < KEEP; ++m) {
+        const int at = r - KEEP + m;                // the row of this input, if the step has it
+#pragma unroll
+        for (int u = 0; u < NQ; ++u) {
+          const int d = 4 * (lane + 32 * u);
+          float x[4] = {0.f, 0.f, 0.f, 0.f};
+          if (d < size)
+            Quad<float>::load(at >= start ? proj + (size_t)at * ld + ch0 + d
+                                          : cs + (size_t)(KEEP + at - start) * dm.channels + ch0 + d,
+                              x);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) past[u][i][m] = x[i];
+        }
+      }
+    }
+    float y[NQ][4];
+    float ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < NQ; ++u) {
+      const int d = 4 * (lane + 32 * u);
+      float x[4] = {0.f, 0.f, 0.f, 0.f};
+      if (d < size) Quad<float>::load(proj + (size_t)r * ld + ch0 + d, x);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        float acc = 0.f;
+#pragma unroll
+        for (int m = 0; m < KEEP; ++m) acc = fmaf(w[u][i][m], past[u][i][m], acc);
+        acc = fmaf(w[u][i][KEEP], x[i], acc);
+        y[u][i] = acc * sigmoid_f(acc);
+        ss += y[u][i] * y[u][i];
+#pragma unroll
+        for (int m = 0; m + 1 < KEEP; ++m) past[u][i][m] = past[u][i][m + 1];
+        if (KEEP > 0) past[u][i][KEEP > 0 ? KEEP - 1 : 0] = x[i];
+      }
+      if (update_state && d < size) {
+#pragma unroll
+        for (int m = 0; m < KEEP; ++m) {
+          const float s4[4] = {past[u][0][m], past[u][1][m], past[u][2][m], past[u][3][m]};
+          Quad<float>::store(cs + (size_t)m * dm.channels + ch0 + d, s4);
+        }
+      }
+    }
+    float f = 1.f;
+    float* dst;
+    if (unit < 2 * G) {
+      const bool is_q = unit < G;
+      ss = warp_sum(ss);
+      f = (is_q ? rsqrtf((float)D) : 1.f) / sqrtf(ss + 1e-6f);
+      dst = (is_q ? qn : kn) + (size_t)r * GD + (size_t)(is_q ? unit : unit - G) * D;
+    } else {
+      dst = v + ((size_t)r * H + (unit - 2 * G)) * Vd;
+    }
+#pragma unroll
+    for (int u = 0; u < NQ; ++u) {
+      const int d = 4 * (lane + 32 * u);
+      if (d < size) {
+        const float o4[4] = {y[u][0] * f, y[u][1] * f, y[u][2] * f, y[u][3] * f};
+        Quad<float>::store(dst + d, o4);
+      }
+    }
   }
 }
 
@@ -149,7 +276,8 @@ __device__ __forceinline__ void copy_async_wait() {
 // (a warp a column, eight columns a block) where they do not (one long prompt): a token is a chain
 // of dependent instructions for a warp, and with eight times the lanes a column the chain is short
 // and eight times as many warps share an SM's schedulers.
-template <int DPER, int LP, int CHUNK, int THREADS>
+// ONE_DECAY: g holds a decay a head; it travels beside beta.
+template <int DPER, int LP, int CHUNK, int THREADS, bool ONE_DECAY>
 __global__ void __launch_bounds__(THREADS)
 delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ kn,
                         const float* __restrict__ v, const float* __restrict__ g,
@@ -157,7 +285,9 @@ delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ 
                         const int* __restrict__ cu_seqlens, const int* __restrict__ slot_ids,
                         DeltaDims dm, float* __restrict__ o) {
   constexpr int Dp = LP * DPER;
-  constexpr int kTok = 3 * Dp + kMaxColumnsPerBlock + 4;      // floats a token in a stage
+  constexpr int kV = (ONE_DECAY ? 2 : 3) * Dp;                 // where a token's v columns start
+  constexpr int kB = kV + kMaxColumnsPerBlock;                 // beta (and the head's decay)
+  constexpr int kTok = kB + 4;                                 // floats a token in a stage
   extern __shared__ __align__(16) float stage[];               // [kStages][CHUNK][kTok]
   constexpr int cols = THREADS / LP;
   const int b = blockIdx.x / dm.H, h = blockIdx.x - b * dm.H;
@@ -181,7 +311,7 @@ delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ 
   const int ncols = min(cols, Vd - col0);
   // 16-byte copies where rows allow it (a thread keeps the same piece of every token), else 4-byte
   const bool vec = (D & 3) == 0 && (Vd & 3) == 0 && (ncols & 3) == 0;
-  const int dq = D >> 2, pieces = 3 * dq + (ncols >> 2);
+  const int dq = D >> 2, nd = (ONE_DECAY ? 2 : 3) * dq, pieces = nd + (ncols >> 2);
   auto ask = [&](int chunk) {                      // the chunk's tokens into stage chunk % kStages
     float* st = stage + (size_t)(chunk % kStages) * CHUNK * kTok;
     const int ta = t0 + chunk * CHUNK, n = min(CHUNK, t1 - ta);
@@ -192,33 +322,39 @@ delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ 
         if (e < dq) src = kn + (size_t)ta * GD + (size_t)kvh * D + 4 * e, dst = 4 * e, step = (int)GD;
         else if (e < 2 * dq)
           src = qn + (size_t)ta * GD + (size_t)kvh * D + 4 * (e - dq), dst = Dp + 4 * (e - dq), step = (int)GD;
-        else if (e < 3 * dq)
+        else if (!ONE_DECAY && e < nd)
           src = g + (size_t)ta * HD + (size_t)h * D + 4 * (e - 2 * dq), dst = 2 * Dp + 4 * (e - 2 * dq),
           step = (int)HD;
         else
-          src = v + (size_t)ta * HV + (size_t)h * Vd + col0 + 4 * (e - 3 * dq),
-          dst = 3 * Dp + 4 * (e - 3 * dq), step = (int)HV;
+          src = v + (size_t)ta * HV + (size_t)h * Vd + col0 + 4 * (e - nd),
+          dst = kV + 4 * (e - nd), step = (int)HV;
         for (int tt = 0; tt < n; ++tt)
           asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(
                            smem_u32(st + (size_t)tt * kTok + dst)),
                        "l"(src + (size_t)tt * step)
                        : "memory");
       }
-      if (threadIdx.x < n)
-        copy_async_4(st + (size_t)threadIdx.x * kTok + 3 * Dp + kMaxColumnsPerBlock,
+      if (threadIdx.x < n) {
+        copy_async_4(st + (size_t)threadIdx.x * kTok + kB,
                      beta + (size_t)(ta + threadIdx.x) * dm.H + h);
+        if (ONE_DECAY)
+          copy_async_4(st + (size_t)threadIdx.x * kTok + kB + 1,
+                       g + (size_t)(ta + threadIdx.x) * dm.H + h);
+      }
     } else {
-      const int per = 3 * D + ncols + 1;
+      const int rd = (ONE_DECAY ? 2 : 3) * D;
+      const int per = rd + ncols + (ONE_DECAY ? 2 : 1);
       for (int i = threadIdx.x; i < n * per; i += blockDim.x) {
         const int tt = i / per, e = i - tt * per;
         const size_t t = (size_t)(ta + tt);
         float* dst = st + (size_t)tt * kTok;
         if (e < D) copy_async_4(dst + e, kn + t * GD + (size_t)kvh * D + e);
         else if (e < 2 * D) copy_async_4(dst + Dp + (e - D), qn + t * GD + (size_t)kvh * D + (e - D));
-        else if (e < 3 * D) copy_async_4(dst + 2 * Dp + (e - 2 * D), g + t * HD + (size_t)h * D + (e - 2 * D));
-        else if (e < 3 * D + ncols)
-          copy_async_4(dst + 3 * Dp + (e - 3 * D), v + t * HV + (size_t)h * Vd + col0 + (e - 3 * D));
-        else copy_async_4(dst + 3 * Dp + kMaxColumnsPerBlock, beta + t * dm.H + h);
+        else if (!ONE_DECAY && e < rd) copy_async_4(dst + 2 * Dp + (e - 2 * D), g + t * HD + (size_t)h * D + (e - 2 * D));
+        else if (e < rd + ncols)
+          copy_async_4(dst + kV + (e - rd), v + t * HV + (size_t)h * Vd + col0 + (e - rd));
+        else if (e == rd + ncols) copy_async_4(dst + kB, beta + t * dm.H + h);
+        else copy_async_4(dst + kB + 1, g + t * dm.H + h);
       }
     }
     copy_async_commit();
@@ -249,12 +385,13 @@ delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ 
         const float* tok = st + (size_t)tt * kTok;
         const float4* k4 = reinterpret_cast<const float4*>(tok + row0);
         const float4* q4 = reinterpret_cast<const float4*>(tok + Dp + row0);
-        const float4* g4 = reinterpret_cast<const float4*>(tok + 2 * Dp + row0);
-        const float vc = tok[3 * Dp + lc], bc = tok[3 * Dp + kMaxColumnsPerBlock];
+        const float4* g4 = reinterpret_cast<const float4*>(tok + 2 * Dp + row0);   // (not ONE_DECAY)
+        const float vc = tok[kV + lc], bc = tok[kB], g1 = tok[kB + 1];
         float kc[DPER];
 #pragma unroll
         for (int i = 0; i < DPER / 4; ++i) {
-          const float4 kk = k4[i], gg = g4[i];
+          const float4 kk = k4[i];
+          const float4 gg = ONE_DECAY ? make_float4(g1, g1, g1, g1) : g4[i];
           kc[4 * i] = kk.x, kc[4 * i + 1] = kk.y, kc[4 * i + 2] = kk.z, kc[4 * i + 3] = kk.w;
           S[4 * i] *= gg.x, S[4 * i + 1] *= gg.y, S[4 * i + 2] *= gg.z, S[4 * i + 3] *= gg.w;
         }
@@ -331,7 +468,7 @@ static DeltaDims dims_of(int H, int G, int D, int Vd, int taps, int state_stride
   DeltaDims dm;
   dm.H = H, dm.G = G, dm.D = D, dm.Vd = Vd, dm.taps = taps;
   dm.channels = 2 * G * D + H * Vd;
-  dm.state_stride = state_stride, dm.conv_off = conv_off;
+  dm.state_stride = state_stride, dm.conv_off = conv_off, dm.a_ld = 0;
   return dm;
 }
 
@@ -351,11 +488,11 @@ GF_EXPORT int gf_delta_prepare(const void* proj, int ld, int b_off, const float*
   const dim3 pgrid(T, (units + kPrepareWarps - 1) / kPrepareWarps), pblock(kPrepareWarps * 32);
   int rc;
   if (dtype == GF_F32)
-    rc = launch_kernel(delta_prepare_kernel<float>, pgrid, pblock, 0, st, (const float*)proj, ld,
+    rc = launch_kernel(delta_prepare_kernel<float, false>, pgrid, pblock, 0, st, (const float*)proj, ld,
                        b_off, a, conv_w, dt_bias, A_log, (const float*)state, seq_of_token,
                        cu_seqlens, slot_ids, dm, qn, kn, v, g, beta);
   else
-    rc = launch_kernel(delta_prepare_kernel<bf>, pgrid, pblock, 0, st, (const bf*)proj, ld, b_off,
+    rc = launch_kernel(delta_prepare_kernel<bf, false>, pgrid, pblock, 0, st, (const bf*)proj, ld, b_off,
                        a, conv_w, dt_bias, A_log, (const float*)state, seq_of_token, cu_seqlens,
                        slot_ids, dm, qn, kn, v, g, beta);
   if (rc || taps == 1) return rc;
@@ -367,10 +504,55 @@ GF_EXPORT int gf_delta_prepare(const void* proj, int ld, int b_off, const float*
                        state, cu_seqlens, slot_ids, dm);
 }
 
+// One decay a head.  proj: [T, ld] fp32 with the columns q | k | v first and the heads' decay
+// pre-activations and betas at a_off and b_off.  max_q_len: the step's longest portion.
+GF_EXPORT int gf_delta_prepare_heads(const float* proj, int ld, int a_off, int b_off,
+                                     const float* conv_w, const float* dt_bias, const float* A_log,
+                                     float* state, const int* seq_of_token, const int* cu_seqlens,
+                                     const int* slot_ids, int T, int B, int max_q_len, int H, int G,
+                                     int D, int Vd, int taps, int state_stride, int conv_off,
+                                     float* qn, float* kn, float* v, float* g, float* beta,
+                                     void* stream) {
+  if (T <= 0) return 0;
+  if (H % G || taps < 1 || D > 32 * kPrepareMaxPerLane) return -3;
+  DeltaDims dm = dims_of(H, G, D, Vd, taps, state_stride, conv_off);
+  dm.a_ld = ld;
+  auto st = (cudaStream_t)stream;
+  const int units = 2 * G + H + 1;
+  const bool al = (((uintptr_t)proj | (uintptr_t)state | (uintptr_t)qn | (uintptr_t)kn |
+                    (uintptr_t)v) & 15) == 0;
+  bool updated = false;
+  int rc = 1;
+  if (D % 4 == 0 && Vd % 4 == 0 && ld % 4 == 0 && state_stride % 4 == 0 && conv_off % 4 == 0 && al &&
+      D <= 256 && Vd <= 256 && taps <= 4) {
+    // few tokens: one each a warp; many: runs, so that a token's inputs are loaded once
+    const int run = T <= 256 ? 1 : 8;
+    updated = max_q_len == 1;
+    const dim3 grid((T + run - 1) / run, (units + 3) / 4), block(128);
+#define GF_GO(TAPS, NQ)                                                                            \
+  if (taps == TAPS && D <= 128 * NQ && Vd <= 128 * NQ && rc == 1)                                  \
+    rc = launch_kernel(delta_prepare_heads_kernel<TAPS, NQ>, grid, block, 0, st, proj, ld, a_off,  \
+                       b_off, conv_w, dt_bias, A_log, state, seq_of_token, cu_seqlens, slot_ids,   \
+                       dm, T, run, updated ? 1 : 0, qn, kn, v, g, beta);
+    GF_GO(1, 1) GF_GO(2, 1) GF_GO(3, 1) GF_GO(4, 1)
+    GF_GO(1, 2) GF_GO(2, 2) GF_GO(3, 2) GF_GO(4, 2)
+#undef GF_GO
+  } else {
+    const dim3 grid(T, (units + kPrepareWarps - 1) / kPrepareWarps), block(kPrepareWarps * 32);
+    rc = launch_kernel(delta_prepare_kernel<float, true>, grid, block, 0, st, proj, ld, b_off,
+                       proj + a_off, conv_w, dt_bias, A_log, (const float*)state, seq_of_token,
+                       cu_seqlens, slot_ids, dm, qn, kn, v, g, beta);
+  }
+  if (rc || taps == 1 || updated) return rc;
+  return launch_kernel(delta_conv_state_kernel<float>, dim3((dm.channels + 127) / 128, B), dim3(128),
+                       0, st, proj, ld, state, cu_seqlens, slot_ids, dm);
+}
+
+// one_decay: g is [T, H] (a decay a head), else [T, H, D].
 GF_EXPORT int gf_delta_recurrence(const float* qn, const float* kn, const float* v, const float* g,
                                   const float* beta, float* state, const int* cu_seqlens,
                                   const int* slot_ids, int B, int H, int G, int D, int Vd,
-                                  int state_stride, float* o, void* stream) {
+                                  int state_stride, float* o, int one_decay, void* stream) {
   if (B <= 0) return 0;
   if (H % G) return -3;
   const DeltaDims dm = dims_of(H, G, D, Vd, 1, state_stride, 0);
@@ -383,12 +565,18 @@ GF_EXPORT int gf_delta_recurrence(const float* qn, const float* kn, const float*
   const int cols = threads / lp;
   const dim3 grid(B * H, (Vd + cols - 1) / cols);
   const dim3 block(threads);
+#define GF_AS(DPER, LP, CHUNK, THREADS, ONE)                                                       \
+  {                                                                                                \
+    const size_t smem =                                                                            \
+        (size_t)kStages * CHUNK * ((ONE ? 2 : 3) * LP * DPER + kMaxColumnsPerBlock + 4) *          \
+        sizeof(float);                                                                             \
+    return launch_kernel(delta_recurrence_kernel<DPER, LP, CHUNK, THREADS, ONE>, grid, block,      \
+                         smem, st, qn, kn, v, g, beta, state, cu_seqlens, slot_ids, dm, o);        \
+  }
 #define GF_GO(DPER, LP, CHUNK, THREADS)                                                            \
   if (lp == LP && D <= LP * DPER) {                                                                \
-    const size_t smem =                                                                            \
-        (size_t)kStages * CHUNK * (3 * LP * DPER + kMaxColumnsPerBlock + 4) * sizeof(float);       \
-    return launch_kernel(delta_recurrence_kernel<DPER, LP, CHUNK, THREADS>, grid, block, smem, st,  \
-                         qn, kn, v, g, beta, state, cu_seqlens, slot_ids, dm, o);                  \
+    if (one_decay) GF_AS(DPER, LP, CHUNK, THREADS, true)                                           \
+    GF_AS(DPER, LP, CHUNK, THREADS, false)                                                         \
   }
   GF_GO(4, 4, 8, kRecurrenceThreads)
   GF_GO(8, 4, 8, kRecurrenceThreads)
@@ -399,6 +587,7 @@ GF_EXPORT int gf_delta_recurrence(const float* qn, const float* kn, const float*
   GF_GO(4, 32, 8, 256)
   GF_GO(8, 32, 4, 256)
 #undef GF_GO
+#undef GF_AS
   return -3;
 }
 

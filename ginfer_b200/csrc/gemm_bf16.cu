@@ -48,9 +48,9 @@
 namespace gf {
 
 constexpr int NTHREADS = 192;
-// EPI_RELU2: EPI_STORE whose result, bias included, passes relu(x)^2 (instances of its own, for
-// the token tiles of decode steps only, so that the plain store keeps its code).
-constexpr int EPI_STORE = 0, EPI_RELU2 = 1, EPI_SILU = 2, EPI_RESID = 3;
+// EPI_RELU2, EPI_XIELU: EPI_STORE whose result, bias included, passes relu(x)^2 or xIELU (instances
+// of their own, for the token tiles of decode steps only, so that the plain store keeps its code).
+constexpr int EPI_STORE = 0, EPI_RELU2 = 1, EPI_SILU = 2, EPI_RESID = 3, EPI_XIELU = 4;
 
 struct GemmExtra {
   // consumer of a deferred RMS normalisation: scale[m] = rsqrt(sum_p in_sumsq[p][m] * inv_k + eps)
@@ -65,10 +65,15 @@ struct GemmExtra {
   const void* gamma;         // [N], bf16 or fp32
   int gamma_f32;
   float* out_sumsq;          // [parts][ss_ld]; part = tile of rows (* splits + split)
+  float act_a, act_b;        // EPI_XIELU
 };
 __device__ __forceinline__ float relu2(float x) {
   x = fmaxf(x, 0.f);
   return x * x;
+}
+template <int EPI>
+__device__ __forceinline__ float activated(float x, const GemmExtra& ex) {
+  return EPI == EPI_RELU2 ? relu2(x) : EPI == EPI_XIELU ? xielu(x, ex.act_a, ex.act_b) : x;
 }
 constexpr int kMaxTiles = 1 << 16;
 __device__ unsigned int g_tile_done[kMaxTiles];
@@ -138,14 +143,13 @@ __device__ __forceinline__ void epilogue16(float (&v)[16], OUT* __restrict__ out
 #pragma unroll
     for (int j = 0; j < 16; ++j) v[j] *= scale[j];
   }
-  if (EPI == EPI_STORE || EPI == EPI_RELU2) {
+  if (EPI == EPI_STORE || EPI == EPI_RELU2 || EPI == EPI_XIELU) {
     const float b = (bias && n < N) ? bias[n] : 0.f;
     if (n < N) {
 #pragma unroll
       for (int j = 0; j < 16; ++j)
         if (m_base + j < M)
-          store_out<OUT>(out + (size_t)(m_base + j) * ldo + n,
-                         EPI == EPI_RELU2 ? relu2(v[j] + b) : v[j] + b);
+          store_out<OUT>(out + (size_t)(m_base + j) * ldo + n, activated<EPI>(v[j] + b, ex));
     }
   } else if (EPI == EPI_RESID) {
     const float b = (bias && n < N) ? bias[n] : 0.f;
@@ -330,9 +334,9 @@ __device__ __forceinline__ void cluster_reduce(uint32_t red, const float* recv, 
                   if (ex.out_scaled) ex.out_scaled[at + j] = __float2bfloat16_rn(g[j]);
                 }
             }
-          } else if (EPI == EPI_RELU2) {
+          } else if (EPI == EPI_RELU2 || EPI == EPI_XIELU) {
 #pragma unroll
-            for (int j = 0; j < 4; ++j) v[j] = relu2(v[j]);
+            for (int j = 0; j < 4; ++j) v[j] = activated<EPI>(v[j], ex);
             if (vec) {
               store4(out + at, v);
             } else {
@@ -856,7 +860,7 @@ static int dispatch_bn(int bn, const CUtensorMap& mw, const CUtensorMap& mx, con
     GF_CASE(32);
     GF_CASE(64);
   }
-  if (EPI != EPI_RESID && EPI != EPI_RELU2) {   // these serve the token tiles of decode steps only
+  if (EPI != EPI_RESID && EPI != EPI_RELU2 && EPI != EPI_XIELU) {   // these serve the token tiles of decode steps only
     switch (bn) {
       GF_CASE(128);
       GF_CASE(256);
@@ -900,7 +904,7 @@ GF_EXPORT long long gf_gemm_bf16_workspace_words(int M, int N, int split_k) {
 // (gate_i, up_i), out[m, i] = silu(gate) * up, N even; epi 3: out (fp32) = resid + acc + bias with
 // out_scaled = bf16(out * gamma[n]) (if given) and out_sumsq[part][m] = the part's share of
 // sum_n out^2, parts = gf_gemm_bf16_parts(N, split_k) rows of ss_ld floats; ldo == N, M <= 64,
-// cluster mode or no split.  out_f32: fp32 output (epi 0, 3).  ldx, ldo in elements.
+// cluster mode or no split; epi 1 / 4: epi 0 through relu(x)^2 / xIELU (act_a, act_b).  out_f32: fp32 output (epi 0, 3).  ldx, ldo in elements.
 // in_sumsq (in_parts rows of ss_ld floats): the accumulator of token m is multiplied by
 // rsqrt(sum_p in_sumsq[p][m] / K + in_eps) before bias and epilogue.
 // split_k > 1 with a workspace: workspace mode; without: cluster mode (split_k 2, 4, 8 or 12).
@@ -915,11 +919,13 @@ GF_EXPORT int gf_gemm_bf16_tc_ex(const void* x, int ldx, const void* w, const fl
                                  int split_k, void* workspace, int* err, void* stream,
                                  const float* in_sumsq, int in_parts, int ss_ld, float in_eps,
                                  const float* resid, void* out_scaled, const void* gamma,
-                                 int gamma_f32, float* out_sumsq) {
+                                 int gamma_f32, float* out_sumsq, float act_a, float act_b) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || K % 8 || ldx % 8 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return -6;
   if (epi == EPI_SILU && ((N & 1) || out_f32)) return -6;
-  if (epi != EPI_STORE && epi != EPI_RELU2 && epi != EPI_SILU && epi != EPI_RESID) return -6;
+  if (epi != EPI_STORE && epi != EPI_RELU2 && epi != EPI_SILU && epi != EPI_RESID &&
+      epi != EPI_XIELU)
+    return -6;
   const int bn = gf_gemm_bf16_token_tile(M);
   if (split_k < 1) split_k = 1;
   if (epi == EPI_RESID) {
@@ -946,6 +952,8 @@ GF_EXPORT int gf_gemm_bf16_tc_ex(const void* x, int ldx, const void* w, const fl
   ex.gamma = gamma;
   ex.gamma_f32 = gamma_f32;
   ex.out_sumsq = out_sumsq;
+  ex.act_a = act_a;
+  ex.act_b = act_b;
   auto st = (cudaStream_t)stream;
   float* ws = (float*)workspace;
   if (epi == EPI_SILU)
@@ -961,6 +969,13 @@ GF_EXPORT int gf_gemm_bf16_tc_ex(const void* x, int ldx, const void* w, const fl
     return dispatch_bn<EPI_RELU2, bf16>(bn, mw, mx, bias, out, ldo, M, N, K, split_k, ws, err, st,
                                         ex);
   }
+  if (epi == EPI_XIELU) {
+    if (out_f32)
+      return dispatch_bn<EPI_XIELU, float>(bn, mw, mx, bias, out, ldo, M, N, K, split_k, ws, err,
+                                           st, ex);
+    return dispatch_bn<EPI_XIELU, bf16>(bn, mw, mx, bias, out, ldo, M, N, K, split_k, ws, err, st,
+                                        ex);
+  }
   if (out_f32)
     return dispatch_bn<EPI_STORE, float>(bn, mw, mx, bias, out, ldo, M, N, K, split_k, ws, err, st,
                                          ex);
@@ -971,5 +986,6 @@ GF_EXPORT int gf_gemm_bf16_tc(const void* x, int ldx, const void* w, const float
                               int ldo, int M, int N, int K, int epi, int out_f32, int split_k,
                               void* workspace, int* err, void* stream) {
   return gf_gemm_bf16_tc_ex(x, ldx, w, bias, out, ldo, M, N, K, epi, out_f32, split_k, workspace,
-                            err, stream, nullptr, 0, 0, 0.f, nullptr, nullptr, nullptr, 0, nullptr);
+                            err, stream, nullptr, 0, 0, 0.f, nullptr, nullptr, nullptr, 0, nullptr,
+                            0.f, 0.f);
 }

@@ -350,6 +350,130 @@ __global__ void qk_norm_rope_vec_kernel(T* __restrict__ qkv, int stride, int num
   }
 }
 
+// Rotation first, then a norm without weights, over heads of hd channels of which norm_dim are real
+// (the rest are zero padding and stay zero).  Pairs (i, i + n_pairs); cosine and sine are multiplied
+// by rot_mult, so the rotated channels are stretched and the norm behind them sees that.  q in place,
+// k to the cache; the values (vd channels a head) go to the cache as they are.
+struct RopeNormDims {
+  int stride, nh, nkv, hd, vd, norm_dim, k_off, v_off, n_pairs;
+  float eps, rot_mult;
+};
+
+// One warp per (token, head).
+template <typename T>
+__global__ void qk_rope_norm_kernel(T* __restrict__ qkv, int num_tokens, const RopeNormDims dm,
+                                    const float* __restrict__ freqs,
+                                    const int* __restrict__ positions,
+                                    const int* __restrict__ slot_mapping, T* __restrict__ kpages,
+                                    T* __restrict__ vpages) {
+  const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+  pdl_trigger();
+  pdl_wait();
+  const int heads = dm.nh + dm.nkv;
+  if (warp >= num_tokens * heads) return;
+  const int t = warp / heads, h = warp - t * heads;
+  const bool is_k = h >= dm.nh;
+  if (is_k && slot_mapping == nullptr) return;
+  const int kh = h - dm.nh, n_pairs = dm.n_pairs;
+  T* src = qkv + (size_t)t * dm.stride + (is_k ? dm.k_off + kh * dm.hd : h * dm.hd);
+  T* dst = src;
+  if (is_k) {
+    const size_t at = (size_t)slot_mapping[t] * dm.nkv + kh;
+    dst = kpages + at * dm.hd;
+    const T* vsrc = qkv + (size_t)t * dm.stride + dm.v_off + kh * dm.vd;
+    for (int c = lane; c < dm.vd; c += 32) vpages[at * dm.vd + c] = vsrc[c];
+  }
+  const float pos = (float)positions[t];
+  float ss = 0.f;
+  for (int i = lane; i < n_pairs; i += 32) {         // a rotated pair keeps its length but for rot_mult
+    const float u = to_f32(src[i]), v = to_f32(src[i + n_pairs]);
+    float sn, cs;
+    sincosf(pos * freqs[i], &sn, &cs);
+    sn *= dm.rot_mult, cs *= dm.rot_mult;
+    const float a = u * cs - v * sn, b = v * cs + u * sn;
+    ss += a * a + b * b;
+  }
+  for (int c = 2 * n_pairs + lane; c < dm.hd; c += 32) {
+    const float u = to_f32(src[c]);
+    ss += u * u;
+  }
+  ss = warp_sum(ss);                                  // (every lane has read its channels)
+  const float inv = 1.f / sqrtf(ss / (float)dm.norm_dim + dm.eps);
+  for (int i = lane; i < n_pairs; i += 32) {
+    const float u = to_f32(src[i]), v = to_f32(src[i + n_pairs]);
+    float sn, cs;
+    sincosf(pos * freqs[i], &sn, &cs);
+    sn *= dm.rot_mult, cs *= dm.rot_mult;
+    dst[i] = from_f32<T>((u * cs - v * sn) * inv);
+    dst[i + n_pairs] = from_f32<T>((v * cs + u * sn) * inv);
+  }
+  for (int c = 2 * n_pairs + lane; c < dm.hd; c += 32) dst[c] = from_f32<T>(to_f32(src[c]) * inv);
+}
+
+// The same for heads of up to 128 channels with hd, vd and n_pairs multiples of 4: a block a token,
+// which takes the angles' sines and cosines once, into shared memory, for all of its heads; a warp a
+// head at a time, a lane owns four neighbouring channels; a pair's other half is another lane's.
+template <typename T>
+__global__ void qk_rope_norm_vec_kernel(T* __restrict__ qkv, const RopeNormDims dm,
+                                        const float* __restrict__ freqs,
+                                        const int* __restrict__ positions,
+                                        const int* __restrict__ slot_mapping,
+                                        T* __restrict__ kpages, T* __restrict__ vpages) {
+  extern __shared__ __align__(16) float tab[];        // cos[n_pairs], sin[n_pairs]
+  const int t = blockIdx.x, lane = threadIdx.x & 31, n_pairs = dm.n_pairs;
+  pdl_trigger();
+  pdl_wait();
+  {
+    const float pos = (float)positions[t];
+    for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) {
+      float sn, cs;
+      sincosf(pos * freqs[i], &sn, &cs);
+      tab[i] = cs * dm.rot_mult;
+      tab[n_pairs + i] = sn * dm.rot_mult;
+    }
+  }
+  __syncthreads();
+  const int heads = slot_mapping ? dm.nh + dm.nkv : dm.nh;
+  const int c = 4 * lane, hq = n_pairs >> 2;          // the pairs' halves are hq lanes apart
+  const bool first = lane < hq, second = !first && lane < 2 * hq;
+  const int other = first ? lane + hq : second ? lane - hq : lane;
+  for (int h = threadIdx.x >> 5; h < heads; h += blockDim.x >> 5) {
+    const bool is_k = h >= dm.nh;
+    const int kh = h - dm.nh;
+    T* src = qkv + (size_t)t * dm.stride + (is_k ? dm.k_off + kh * dm.hd : h * dm.hd);
+    T* dst = src;
+    float x[4] = {0.f, 0.f, 0.f, 0.f}, y[4];
+    if (c < dm.hd) Quad<T>::load(src + c, x);
+    if (is_k) {
+      const size_t at = (size_t)slot_mapping[t] * dm.nkv + kh;
+      dst = kpages + at * dm.hd;
+      if (c < dm.vd) {
+        float v[4];
+        Quad<T>::load(qkv + (size_t)t * dm.stride + dm.v_off + kh * dm.vd + c, v);
+        Quad<T>::store(vpages + at * dm.vd + c, v);
+      }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      y[i] = __shfl_sync(0xffffffffu, x[i], other);
+      if (first || second) {
+        const int p = first ? c + i : c + i - n_pairs;
+        const float cs = tab[p], sn = tab[n_pairs + p];
+        x[i] = first ? x[i] * cs - y[i] * sn : x[i] * cs + y[i] * sn;
+      }
+      ss += x[i] * x[i];
+    }
+    ss = warp_sum(ss);
+    const float inv = 1.f / sqrtf(ss / (float)dm.norm_dim + dm.eps);
+    if (c < dm.hd) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) x[i] *= inv;
+      Quad<T>::store(dst + c, x);
+    }
+  }
+}
+
 // Eight channels a thread (hd % 8 == 0, 16-byte aligned rows).
 __global__ void head_gate_vec_kernel(__nv_bfloat16* __restrict__ o,
                                      const __nv_bfloat16* __restrict__ g, int g_stride, int nh,
@@ -508,6 +632,41 @@ GF_EXPORT int gf_qk_norm_rope(void* qkv, int stride, int T, int nh, int nkv, int
   return launch_kernel(qk_norm_rope_kernel<bf>, grid, block, 0, st, (bf*)qkv, stride, T, nh, nkv,
                        hd, k_off, v_off, qw, kw, eps, qt_coef, qt_every, freqs, n_pairs, interleaved, positions,
                        slot_mapping, (bf*)kpages, (bf*)vpages);
+}
+
+// See RopeNormDims.  freqs [n_pairs] or null with n_pairs 0; kpages [.., nkv, hd], vpages
+// [.., nkv, vd]; slot_mapping null: nothing is cached.
+GF_EXPORT int gf_qk_rope_norm(void* qkv, int stride, int T, int nh, int nkv, int hd, int vd,
+                              int norm_dim, int k_off, int v_off, float eps, const float* freqs,
+                              int n_pairs, float rot_mult, const int* positions,
+                              const int* slot_mapping, void* kpages, void* vpages, int dtype,
+                              void* stream) {
+  if (T <= 0) return 0;
+  if (2 * n_pairs > norm_dim || norm_dim > hd || norm_dim <= 0 || (n_pairs > 0 && !freqs)) return -3;
+  auto st = (cudaStream_t)stream;
+  const RopeNormDims dm{stride, nh, nkv, hd, vd, norm_dim, k_off, v_off, n_pairs, eps, rot_mult};
+  const int esz = dtype == GF_F32 ? 4 : 2;
+  const bool vec = n_pairs % 4 == 0 && hd % 4 == 0 && vd % 4 == 0 && hd <= 128 && vd <= 128 &&
+                   stride % 4 == 0 && k_off % 4 == 0 && v_off % 4 == 0 &&
+                   (((uintptr_t)qkv | (uintptr_t)kpages | (uintptr_t)vpages) % (4 * esz)) == 0;
+  if (vec) {
+    // few tokens: a warp a head, so that no warp walks over several heads one after the other
+    const int hw = nh + nkv < 16 ? nh + nkv : 16;
+    const dim3 grid(T), block(T <= 256 ? 32 * hw : 128);
+    const size_t smem = 2 * (size_t)n_pairs * sizeof(float);
+    if (dtype == GF_F32)
+      return launch_kernel(qk_rope_norm_vec_kernel<float>, grid, block, smem, st, (float*)qkv, dm,
+                           freqs, positions, slot_mapping, (float*)kpages, (float*)vpages);
+    return launch_kernel(qk_rope_norm_vec_kernel<bf>, grid, block, smem, st, (bf*)qkv, dm, freqs,
+                         positions, slot_mapping, (bf*)kpages, (bf*)vpages);
+  }
+  const size_t warps = (size_t)T * (nh + nkv);
+  const dim3 grid((unsigned)((warps + 3) / 4)), block(128);
+  if (dtype == GF_F32)
+    return launch_kernel(qk_rope_norm_kernel<float>, grid, block, 0, st, (float*)qkv, T, dm, freqs,
+                         positions, slot_mapping, (float*)kpages, (float*)vpages);
+  return launch_kernel(qk_rope_norm_kernel<bf>, grid, block, 0, st, (bf*)qkv, T, dm, freqs,
+                       positions, slot_mapping, (bf*)kpages, (bf*)vpages);
 }
 
 GF_EXPORT int gf_head_gate(void* o, const void* g, int g_stride, int T, int nh, int hd, int dtype,

@@ -265,8 +265,8 @@ class ModelRunner:
             decode_only=facts["max_q_len"] == 1, all_rows_wanted=facts["all_rows"])
 
     def binder(self, dev: dict[str, torch.Tensor]):
-        def bind(entry):
-            cid = entry.cache
+        def bind(entry, block=False):
+            cid = entry.block_state if block else entry.cache
             if self.storage.is_paged(cid):
                 g = self.storage.group_of(cid)
                 return PagedKVBinding(self.storage.pages_of(cid), dev[f"block_table{g}"],
@@ -274,7 +274,7 @@ class ModelRunner:
                                       self.groups[g].window, entry.write_cache,
                                       self.groups[g].chunk)
             if cid in self.storage.state:
-                return StateBinding(self.storage.state[cid], entry.write_cache)
+                return StateBinding(self.storage.state[cid], block or entry.write_cache)
             return None
         return bind
 

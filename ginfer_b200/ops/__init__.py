@@ -278,14 +278,15 @@ def silu_mul(gate_up: torch.Tensor) -> torch.Tensor:
     return out
 
 
-def activation_(x: torch.Tensor, kind: str, c: float = 0.0) -> torch.Tensor:
+def activation_(x: torch.Tensor, kind: str, c: float = 0.0, c2: float = 0.0) -> torch.Tensor:
     """In place, fp32 arithmetic: ``kind`` ``"relu2"``: ``relu(x)^2``; ``"softcap"``:
-    ``c * tanh(x / c)``."""
+    ``c * tanh(x / c)``; ``"xielu"``: ``c x^2 + x/2`` above zero, ``c2 (e^x - 1 - x) + x/2`` below."""
     _cuda(x)
     assert x.is_contiguous()
     f = _fn("elementwise", "gf_activation",
-            [c_void_p, c_longlong, c_int, c_float, c_int, c_void_p])
-    rc = f(_p(x), x.numel(), {"relu2": 0, "softcap": 1}[kind], float(c), _code(x.dtype), _stream())
+            [c_void_p, c_longlong, c_int, c_float, c_float, c_int, c_void_p])
+    rc = f(_p(x), x.numel(), {"relu2": 0, "softcap": 1, "xielu": 2}[kind], float(c), float(c2),
+           _code(x.dtype), _stream())
     if rc == -3:
         raise ValueError(f"activation {kind!r} with constant {c}")
     _ok(rc, "activation")
@@ -303,11 +304,13 @@ def mask_span(window: int = 0, chunk: int = 0) -> int:
 
 
 def paged_attention_simt(qkv, pages, block_table, seq_of_token, positions, nh, nkv, hd, scale,
-                         window, page_size, vd=None, softcap: float = 0.0, slopes=None):
+                         window, page_size, vd=None, softcap: float = 0.0, slopes=None,
+                         sink: float | None = None):
     """``window``: the mask as :func:`mask_span` gives it.  ``vd``: the values' head size where
     it is not the keys' (``pages`` is then a pair of tensors).  ``softcap`` > 0: scores pass
     ``cap * tanh(s / cap)``; ``slopes`` (fp32, a head): ``slope * (p - c)`` is taken off the score
-    of the key at ``c`` for the query at ``p``, after the cap."""
+    of the key at ``c`` for the query at ``p``, after the cap; ``sink``: ``exp(sink)`` is added to the
+    softmax's denominator (a score without a key and a value)."""
     _cuda(qkv, pages[0], pages[1], block_table, seq_of_token, positions, slopes)
     assert slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == nh
                               and slopes.is_contiguous())
@@ -316,12 +319,12 @@ def paged_attention_simt(qkv, pages, block_table, seq_of_token, positions, nh, n
     out = torch.empty((T, nh * vd), dtype=qkv.dtype, device=qkv.device)
     f = _fn("attention_simt", "gf_paged_attention_simt",
             [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
-             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int,
-             c_void_p])
+             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_float,
+             c_int, c_void_p])
     rc = f(_p(qkv), qkv.stride(0), _p(pages[0]), _p(pages[1]), _p(block_table),
            block_table.stride(0), _p(seq_of_token), _p(positions), _p(out), T, nh, nkv, hd, vd,
            page_size, int(window), float(scale), float(softcap or 0.0), _p(slopes),
-           _code(qkv.dtype), _stream())
+           float("-inf") if sink is None else float(sink), _code(qkv.dtype), _stream())
     if rc == -3:
         raise ValueError(f"attention kernels take head sizes up to 256 and head counts that are "
                          f"a multiple of the kv head count; got head_dim={hd}, heads={nh}, "
@@ -340,17 +343,17 @@ def attention_fuses_rope(qkv: torch.Tensor, ctx, nh: int, nkv: int, hd: int) -> 
 def paged_attention(qkv: torch.Tensor, pages, block_table: torch.Tensor, ctx,
                     nh: int, nkv: int, hd: int, scale: float, window: int, page_size: int,
                     rope=None, vd: int | None = None, softcap: float = 0.0,
-                    slopes=None) -> torch.Tensor:
+                    slopes=None, sink: float | None = None) -> torch.Tensor:
     """Attention of the step's queries (first ``nh * hd`` columns of ``qkv``) over the paged
     cache; returns ``[T, nh * hd]``.  Picks the kernel by dtype, head size and batch shape.
     ``rope = (table or None, rotary_dim, write)`` where :func:`attention_fuses_rope`: q and k are
     still unrotated and the new k and v not yet in the cache.  ``window``: the mask as
     :func:`mask_span` gives it.  ``vd``: the values' head size if it differs from ``hd``
     (``pages`` is then the pair of the cache's two planes; the result is ``[T, nh * vd]``).
-    ``softcap``, ``slopes``: a soft cap on the scores and a distance bias a head, see
+    ``softcap``, ``slopes``, ``sink``: a soft cap on the scores, a distance bias a head and a sink, see
     :func:`paged_attention_simt`."""
     from . import attention_bf16
-    shaped = dict(softcap=float(softcap or 0.0), slopes=slopes)
+    shaped = dict(softcap=float(softcap or 0.0), slopes=slopes, sink=sink)
     if vd is not None and vd != hd:        # keys and values of different widths: the plain kernel
         assert rope is None
         return paged_attention_simt(qkv, pages, block_table, ctx.seq_of_token, ctx.positions, nh,
@@ -441,4 +444,4 @@ def bmm_f32_out(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
 
 from .linear import GatedLinear, Linear, add_to  # noqa: E402,F401
 from . import prenorm  # noqa: E402,F401
-from . import depth  # noqa: E402,F401
+from . import depth, shift  # noqa: E402,F401

@@ -1,4 +1,4 @@
-"""Gated delta rule with a decay per key channel over per-request state
+"""Gated delta rule with a decay per key channel or per head over per-request state
 (``csrc/delta_rule.cu``)."""
 from __future__ import annotations
 
@@ -7,6 +7,9 @@ from ctypes import c_float, c_int, c_void_p
 import torch
 
 from . import _code, _cuda, _fn, _ok, _p, _stream
+
+
+MAX_KEY_SIZE = 256        # the recurrence kernel's largest
 
 
 def prepare(proj: torch.Tensor, b_off: int, a: torch.Tensor, conv_w: torch.Tensor,
@@ -44,17 +47,53 @@ def prepare(proj: torch.Tensor, b_off: int, a: torch.Tensor, conv_w: torch.Tenso
     return qn, kn, v, g, beta
 
 
+def prepare_heads(proj: torch.Tensor, a_off: int, b_off: int, conv_w: torch.Tensor,
+                  dt_bias: torch.Tensor, A_log: torch.Tensor, state: torch.Tensor, ctx, H: int,
+                  G: int, D: int, Vd: int, taps: int, conv_off: int):
+    """The same with one decay a head: ``proj [T, >= 2 G D + H Vd + ...]`` fp32 holds the q | k | v
+    projections first, the heads' decay pre-activations at ``a_off`` and the beta columns at
+    ``b_off``.  Returns fp32 ``(q [T, G, D], k [T, G, D], v [T, H, Vd], g [T, H], beta [T, H])``."""
+    _cuda(proj, conv_w, dt_bias, A_log, state)
+    T = proj.shape[0]
+    assert proj.dim() == 2 and proj.stride(1) == 1 and proj.dtype == torch.float32
+    assert max(a_off, b_off) + H <= proj.shape[1]
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous()
+    ch = 2 * G * D + H * Vd
+    assert conv_w.dtype == torch.float32 and conv_w.shape == (ch, taps) and conv_w.is_contiguous()
+    assert dt_bias.dtype == torch.float32 and dt_bias.numel() == H
+    assert A_log.dtype == torch.float32 and A_log.numel() == H
+    dev = proj.device
+    qn = torch.empty((T, G, D), dtype=torch.float32, device=dev)
+    kn = torch.empty_like(qn)
+    v = torch.empty((T, H, Vd), dtype=torch.float32, device=dev)
+    g = torch.empty((T, H), dtype=torch.float32, device=dev)
+    beta = torch.empty_like(g)
+    f = _fn("delta_rule", "gf_delta_prepare_heads",
+            [c_void_p, c_int, c_int, c_int] + [c_void_p] * 7 + [c_int] * 10 + [c_void_p] * 6)
+    rc = f(_p(proj), proj.stride(0), int(a_off), int(b_off), _p(conv_w), _p(dt_bias), _p(A_log),
+           _p(state), _p(ctx.seq_of_token), _p(ctx.cu_seqlens_q), _p(ctx.slot_ids), T,
+           ctx.num_seqs, int(ctx.max_q_len), H, G, D, Vd, taps, state.stride(0), int(conv_off),
+           _p(qn), _p(kn), _p(v), _p(g), _p(beta), _stream())
+    if rc == -3:
+        raise ValueError("the delta-rule kernels need heads to be a multiple of kv heads and key "
+                         f"sizes up to {MAX_KEY_SIZE}; got {H} heads, {G} kv heads, key size {D}")
+    _ok(rc, "delta_prepare_heads")
+    return qn, kn, v, g, beta
+
+
 def recurrence(qn, kn, v, g, beta, state: torch.Tensor, ctx) -> torch.Tensor:
-    """Advance every request's state over its tokens of this step; returns ``o [T, H, Vd]`` fp32."""
+    """Advance every request's state over its tokens of this step; returns ``o [T, H, Vd]`` fp32.
+    ``g``: ``[T, H, D]``, or ``[T, H]`` for one decay a head."""
     T, G, D = qn.shape
     H, Vd = v.shape[1], v.shape[2]
     o = torch.empty((T, H, Vd), dtype=torch.float32, device=qn.device)
     f = _fn("delta_rule", "gf_delta_recurrence",
-            [c_void_p] * 8 + [c_int] * 6 + [c_void_p, c_void_p])
+            [c_void_p] * 8 + [c_int] * 6 + [c_void_p, c_int, c_void_p])
     rc = f(_p(qn), _p(kn), _p(v), _p(g), _p(beta), _p(state), _p(ctx.cu_seqlens_q),
-           _p(ctx.slot_ids), ctx.num_seqs, H, G, D, Vd, state.stride(0), _p(o), _stream())
+           _p(ctx.slot_ids), ctx.num_seqs, H, G, D, Vd, state.stride(0), _p(o), int(g.dim() == 2),
+           _stream())
     if rc == -3:
-        raise ValueError(f"the delta-rule recurrence takes key sizes up to 256, got {D}")
+        raise ValueError(f"the delta-rule recurrence takes key sizes up to {MAX_KEY_SIZE}, got {D}")
     _ok(rc, "delta_recurrence")
     return o
 

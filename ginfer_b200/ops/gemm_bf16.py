@@ -110,9 +110,11 @@ def sumsq_ld(M: int) -> int:
 
 
 def gemm(x, weight, bias_f32=None, out_dtype=torch.bfloat16, epi: int = 0, split_k=None,
-         through_workspace: bool = False, scale: RowScale | None = None, resid=None, gamma=None):
+         through_workspace: bool = False, scale: RowScale | None = None, resid=None, gamma=None,
+         act_consts=None):
     """``x [M, K] @ weight[N, K]^T``; ``epi`` 0: (+ bias) -> ``[M, N]``; ``epi`` 1: the same
-    through ``relu(.)^2``; ``epi`` 2: weight rows
+    through ``relu(.)^2``; ``epi`` 4: the same through xIELU with ``act_consts = (a, b)`` (``a z^2 +
+    z/2`` above zero, ``b (e^z - 1 - z) + z/2`` below); ``epi`` 2: weight rows
     are interleaved (gate_i, up_i) and the result is ``silu(gate) * up`` -> ``[M, N / 2]``.
     ``split_k``: None picks it; 2, 4, 8 or 12 add up inside a cluster; with ``through_workspace``
     any number of splits adds up through global memory.  ``scale``: the accumulator of every token
@@ -156,11 +158,13 @@ def gemm(x, weight, bias_f32=None, out_dtype=torch.bfloat16, epi: int = 0, split
     f = _fn("gemm_bf16", "gf_gemm_bf16_tc_ex",
             [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
              c_int, c_int, c_void_p, c_void_p, c_void_p,
-             c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
+             c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+             c_float, c_float])
     rc = f(_p(x), x.stride(0), _p(weight), _p(bias_f32), _p(out), cols, M, N, K, int(epi),
            1 if out_dtype == torch.float32 else 0, sk, _p(ws), _p(st["err"]), _stream(),
            _p(in_sumsq), in_parts, ld, in_eps, _p(resid), _p(scaled), _p(gamma),
-           1 if gamma is not None and gamma.dtype == torch.float32 else 0, _p(sumsq))
+           1 if gamma is not None and gamma.dtype == torch.float32 else 0, _p(sumsq),
+           *(float(c) for c in (act_consts or (0.0, 0.0))))
     if rc in (-6, -7):
         return None
     _ok(rc, "gemm_bf16_tc")
@@ -186,13 +190,17 @@ def plain_limit(weight) -> int:
     return PLAIN_MAX_TOKENS_LONG_K if weight.shape[1] >= LONG_K else PLAIN_MAX_TOKENS
 
 
-def try_linear(x, weight, bias_f32, out_dtype, relu2: bool = False):
+_ACTIVATION_EPILOGUES = {None: 0, "relu2": 1, "xielu": 4}
+
+
+def try_linear(x, weight, bias_f32, out_dtype, activation: str | None = None, act_consts=None):
     """Run the tcgen05 kernel where it is the faster one (the small batches of decode steps and
-    short prompt portions); ``None`` hands the product to cuBLAS.  ``relu2``: the result passes
-    ``relu(.)^2`` in the kernel's epilogue."""
+    short prompt portions); ``None`` hands the product to cuBLAS.  ``activation``: the
+    result passes it in the kernel's epilogue (see :func:`gemm`)."""
     if x.shape[0] > plain_limit(weight):
         return None
-    return gemm(x, weight, bias_f32, out_dtype, epi=1 if relu2 else 0)
+    return gemm(x, weight, bias_f32, out_dtype, epi=_ACTIVATION_EPILOGUES[activation],
+                act_consts=act_consts)
 
 
 # Plain products leave for cuBLAS above this many tokens.  In a CUDA graph on a B200, 1.5B shapes,

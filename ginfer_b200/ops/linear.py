@@ -34,15 +34,20 @@ def gemm_f32(x: torch.Tensor, w: torch.Tensor, bias=None) -> torch.Tensor:
 
 class Linear:
     """``y = x W^T + b``.  ``out_dtype`` float32 asks for fp32 results from bf16 operands (the
-    output head).  ``activation="relu2"``: ``y = relu(x W^T + b)^2``, in the product's epilogue
-    where the tcgen05 kernel runs it (few tokens), else in a kernel behind the library's."""
+    output head).  ``activation``: the product passes ``"relu2"`` (``relu(.)^2``) or ``"xielu"``
+    (``act_consts = (a, b)``: ``a z^2 + z/2`` above zero, ``b (e^z - 1 - z) + z/2`` below), in the
+    product's epilogue where the tcgen05 kernel runs it (few tokens), else in a kernel behind the
+    library's."""
 
     def __init__(self, weight: torch.Tensor, bias: torch.Tensor | None = None,
-                 out_dtype: torch.dtype | None = None, activation: str | None = None):
+                 out_dtype: torch.dtype | None = None, activation: str | None = None,
+                 act_consts: tuple[float, float] | None = None):
         _cuda(weight, bias)
-        if activation not in (None, "relu2"):
-            raise ValueError(f"activation {activation!r}: only 'relu2' is there")
-        self.activation = activation
+        if activation not in (None, "relu2", "xielu"):
+            raise ValueError(f"activation {activation!r}: 'relu2' and 'xielu' are there")
+        if (activation == "xielu") != (act_consts is not None):
+            raise ValueError("'xielu' takes two constants, other activations none")
+        self.activation, self.act_consts = activation, act_consts
         self.weight = weight.contiguous()
         self.bias = bias
         self.out_features, self.in_features = weight.shape
@@ -64,11 +69,12 @@ class Linear:
         if (self.dtype == torch.bfloat16 and not hasattr(x, "materialize")
                 and x.dtype == self.dtype):
             from . import gemm_bf16
-            y = gemm_bf16.try_linear(x, self.weight, self._bias_f32, self.out_dtype, relu2=True)
+            y = gemm_bf16.try_linear(x, self.weight, self._bias_f32, self.out_dtype,
+                                     activation=self.activation, act_consts=self.act_consts)
             if y is not None:
                 return y
         from . import activation_
-        return activation_(self._product(x), self.activation)
+        return activation_(self._product(x), self.activation, *(self.act_consts or ()))
 
     def deferring_bias(self, x):
         """``(y, b)`` with ``self(x) = y + b``: ``b`` is the fp32 bias where adding it would cost a

@@ -96,6 +96,30 @@ def qk_norm_rope(qkv: torch.Tensor, nh: int, nkv: int, hd: int, k_off: int, v_of
         "qk_norm_rope")
 
 
+def qk_rope_norm(qkv: torch.Tensor, nh: int, nkv: int, hd: int, vd: int, norm_dim: int, k_off: int,
+                 v_off: int, eps: float, freqs, rot_mult: float, positions: torch.Tensor,
+                 slot_mapping, kpages: torch.Tensor, vpages: torch.Tensor) -> None:
+    """Per head of ``qkv [T, ...]`` (q heads of ``hd`` channels from column 0, k heads from
+    ``k_off``): rotation of the pairs ``(i, i + len(freqs))`` by ``position * freqs[i]`` with cosine
+    and sine times ``rot_mult``, then ``x / sqrt(sum(x^2) / norm_dim + eps)`` (channels from
+    ``norm_dim`` on are zero padding); q in place; with ``slot_mapping`` k goes to ``kpages`` and the
+    values (``vd`` channels a head from ``v_off``, unchanged) to ``vpages``."""
+    _cuda(qkv, freqs, positions, slot_mapping, kpages, vpages)
+    assert qkv.dim() == 2 and qkv.stride(1) == 1
+    assert kpages.is_contiguous() and vpages.is_contiguous()
+    assert kpages.dtype == qkv.dtype and vpages.dtype == qkv.dtype
+    assert tuple(kpages.shape[-2:]) == (nkv, hd) and tuple(vpages.shape[-2:]) == (nkv, vd)
+    n_pairs = 0 if freqs is None else freqs.numel()
+    if freqs is not None:
+        assert freqs.dtype == torch.float32 and freqs.is_contiguous()
+    f = _fn("prenorm_stream", "gf_qk_rope_norm",
+            [c_void_p] + [c_int] * 9 + [c_float, c_void_p, c_int, c_float] + [c_void_p] * 4
+            + [c_int, c_void_p])
+    _ok(f(_p(qkv), qkv.stride(0), qkv.shape[0], nh, nkv, hd, vd, int(norm_dim), int(k_off),
+          int(v_off), float(eps), _p(freqs), n_pairs, float(rot_mult), _p(positions),
+          _p(slot_mapping), _p(kpages), _p(vpages), _code(qkv.dtype), _stream()), "qk_rope_norm")
+
+
 def head_gate(o: torch.Tensor, gates: torch.Tensor, nh: int, hd: int) -> torch.Tensor:
     """``o [T, nh * hd]`` in place: head ``h`` times ``sigmoid(gates[t, h])`` (``gates`` a view
     with any row stride)."""

@@ -166,6 +166,17 @@ class PairSum:
     materialize: Callable[[], torch.Tensor]
 
 
+@dataclass
+class ShiftedInput:
+    """What the first sublayer of a run reads, where that is a norm of the stream shifted towards
+    the token before: ``n_t + (n_(t-1) - n_t) * weight`` with ``n = norm(x)`` and ``weight`` fp32
+    ``[H]``; ``state`` holds ``n`` of the last token of earlier steps, a row a slot.  It takes the
+    place of the plain norm where another block prepares a run's input (``then``)."""
+    norm: "Norm"
+    weight: torch.Tensor
+    state: StateBinding
+
+
 # ----------------------------------------------------------------------------- part interfaces
 class Part:
     """Base of every part."""
@@ -254,6 +265,8 @@ class Block(Part):
     # A block that sets this takes the keyword ``then``: the norm that will consume its output
     # (the next run's first norm), so that its last product can prepare that norm's input.
     takes_next_norm = False
+    # ``then`` may be a :class:`ShiftedInput`
+    prepares_shifted_input = False
 
     def forward(self, x: torch.Tensor, delta: torch.Tensor | None, ctx: StepContext, cache
                 ) -> tuple[torch.Tensor, torch.Tensor | None]:
@@ -262,6 +275,15 @@ class Block(Part):
     def first_norm(self) -> "Norm | None":
         """The norm this block applies to its input first, if another block may prepare it."""
         return None
+
+    # A block that keeps per-request state of its own (beside its mixer's) says what it needs, and
+    # its ``forward`` takes the keyword ``own_state`` (a :class:`StateBinding`).
+    def state_spec(self) -> StateSpec | None:
+        return None
+
+    def first_input(self, own_state: StateBinding | None) -> "Norm | ShiftedInput | None":
+        """What another block may prepare for this one, given the binding of its own state."""
+        return self.first_norm()
 
 
 class StreamInput(Part):

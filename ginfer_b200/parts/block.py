@@ -11,7 +11,7 @@ import os
 
 import torch
 
-from .base import Block, Summed, make_part, register_block
+from .base import Block, ShiftedInput, StateSpec, Summed, make_part, register_block
 
 # Steps of at most this many tokens (bfloat16) fold the additions and normalisations into the
 # neighbouring products: the product before a norm leaves the sum, its product with the norm's
@@ -320,14 +320,19 @@ class SandwichBlock(Block):
     embedding, whose output is state 0) and what goes on to the next layer is ``sum_j w[j] *
     state_j`` over ``j < n`` with the layer's tensor ``depth_name`` (``n`` weights, 32-bit).
 
+    ``shift_name``: the mixer reads its normed input shifted towards the token before, ``n_t +
+    (n_(t-1) - n_t) * w`` with the layer's tensor ``shift_name`` (``w``, 32-bit); the ``n`` of a
+    sequence's last token is the block's own per-request state (``own_state``, zero at the start).
+
     Every sublayer ends in ONE kernel: output norm, addition, (average,) and the norm in front of
-    the next sublayer, also the first norm of the NEXT run (``then``), which travels there in
-    ``ctx.extras["prenormed"]``."""
+    the next sublayer, also the first norm of the NEXT run (``then``; with its shift, if it has
+    one), which travels there in ``ctx.extras["prenormed"]``."""
 
     takes_next_norm = True
+    prepares_shifted_input = True
 
     def __init__(self, layer_spec, mixer_out_norm, feed_forward_out_norm=None,
-                 depth_states: int = 0, depth_name: str = "dwa"):
+                 depth_states: int = 0, depth_name: str = "dwa", shift_name: str | None = None):
         self.spec = layer_spec
         self.mixer_norm = make_part("norm", layer_spec.mixer_norm)
         self.mixer = make_part("mixer", layer_spec.mixer)
@@ -345,6 +350,7 @@ class SandwichBlock(Block):
         if self.depth_states == 1 or self.depth_states < 0:
             raise ValueError("an average over the depth takes at least two states")
         self.depth_w = None
+        self.shift_name, self.shift_w = shift_name, None
 
     def parts(self):
         return tuple(p for p in (self.mixer_norm, self.mixer, self.mixer_out_norm,
@@ -358,6 +364,8 @@ class SandwichBlock(Block):
             out.extend(p.tensor_specs())
         if self.depth_states:
             out.append(TensorSpec(self.depth_name, (self.depth_states,), "f32"))
+        if self.shift_name:
+            out.append(TensorSpec(self.shift_name, (self.mixer_norm.size,), "f32"))
         return out
 
     def first_norm(self):
@@ -368,11 +376,33 @@ class SandwichBlock(Block):
             p.load(tensors, dtype, device)
         if self.depth_states:
             self.depth_w = tensors[self.depth_name].float().contiguous()
+        if self.shift_name:
+            self.shift_w = tensors[self.shift_name].float().contiguous()
+
+    def state_spec(self):
+        return StateSpec((self.mixer_norm.size,), torch.float32) if self.shift_name else None
+
+    def first_input(self, own_state):
+        if not self.shift_name:
+            return self.mixer_norm
+        return ShiftedInput(self.mixer_norm, self.shift_w, own_state)
+
+    def _prepared_here(self, prepared, own_state) -> bool:
+        """Whether what another block prepared is this run's first input."""
+        if isinstance(prepared, ShiftedInput):
+            return prepared.norm is self.mixer_norm and own_state is not None \
+                and prepared.state.state is own_state.state
+        return prepared is self.mixer_norm and not self.shift_name
 
     def _end(self, x, y, out_norm, ctx, nxt, average=False, y_bias=None):
         """One sublayer's end -> ``(stream, norm of the stream for ``nxt`` or None)``.  ``y_bias``:
         a bias the sublayer left for this kernel to add to its output."""
-        from ..ops import depth
+        from ..ops import depth, shift
+        if isinstance(nxt, ShiftedInput) and not (average and self.depth_states) \
+                and y_bias is None and hasattr(nxt.norm, "weight32") and not nxt.norm.weight_offset:
+            return shift.norm_shift(x, ctx.dtype, nxt.norm.weight32(), nxt.norm.eps, nxt.weight,
+                                    nxt.state.state, ctx, y=y, gamma_b=out_norm.weight32(),
+                                    eps_b=out_norm.eps)
         kw = {"y_bias": y_bias} if y_bias is not None else {}
         if average and self.depth_states:
             hist = ctx.extras.get("depth_history")
@@ -380,6 +410,8 @@ class SandwichBlock(Block):
                 raise RuntimeError("this layer averages over the depth, but the step has no "
                                    "history of that many states (the embedding makes it)")
             kw.update(history=hist, mix_weights=self.depth_w, n_before=self.depth_states - 1)
+        if isinstance(nxt, ShiftedInput):        # the next run forms its input itself
+            nxt = None
         fused = nxt is not None and hasattr(nxt, "weight32") and not nxt.weight_offset
         if fused:
             kw.update(next_weight=nxt.weight32(), next_eps=nxt.eps)
@@ -388,14 +420,18 @@ class SandwichBlock(Block):
             n = nxt.forward(x, None, want_sum=False, out_dtype=ctx.dtype)[1]
         return x, n
 
-    def forward(self, x, delta, ctx, cache, then=None):
+    def forward(self, x, delta, ctx, cache, then=None, own_state=None):
         if delta is not None:
             x = x.float() + delta.float()
         elif x.dtype != torch.float32:
             x = x.float()
         kept = ctx.extras.pop("prenormed", None)
-        if kept is not None and kept[0] is x and kept[1] is self.mixer_norm:
+        if kept is not None and kept[0] is x and self._prepared_here(kept[1], own_state):
             n = kept[2]
+        elif self.shift_name:
+            from ..ops import shift
+            n = shift.norm_shift(x, ctx.dtype, self.mixer_norm.weight32(), self.mixer_norm.eps,
+                                 self.shift_w, own_state.state, ctx)[1]
         else:
             n = self.mixer_norm.forward(x, None, want_sum=False, out_dtype=ctx.dtype)[1]
         a = self.mixer.forward(n, ctx, cache)

@@ -1,4 +1,7 @@
-"""Gated delta rule with one decay per head and key channel.
+"""Gated delta rule, with one decay per head and key channel (``channel_delta``) or one per head
+(``head_delta``).
+
+The first:
 
 ``q = W_q h``, ``k = W_k h`` (``G`` kv heads of ``D``), ``v = W_v h`` (``H`` heads of ``Vd``); head
 ``n`` reads q/k head ``n // (H / G)``.  Each passes a short causal convolution over time per
@@ -11,13 +14,16 @@ heads), gated by ``sigmoid(W_g2 (W_g1 h))`` and projected by ``W_o``.
 State per request (one fp32 row of a slot): ``S [H, D, Vd]``, then the last ``taps - 1`` inputs of
 the convolutions ``[taps - 1, 2 G D + H Vd]``.  Decays, gates of the recurrence, unit norms and the
 state are fp32 in both paths.
+
+The second differs in its decay, ``g = exp(-exp(A_log_n) * softplus(W_a h + dt_bias_n))``, a number a
+head, and its gate, ``silu(W_g h)`` with a full matrix.
 """
 from __future__ import annotations
 
 import torch
 
 from .. import ops
-from ..ops import delta
+from ..ops import decay, delta
 from .base import Mixer, StateSpec, TensorSpec, register_mixer
 
 
@@ -97,3 +103,75 @@ class ChannelDelta(Mixer):
 
 
 register_mixer("channel_delta", ChannelDelta)
+
+
+class HeadDelta(Mixer):
+    """The delta rule with one decay a head and a SiLU gate (see the module's text).  One product
+    for everything that reads ``h``, leaving in fp32: its columns feed decays and step sizes, and
+    the convolutions keep their inputs in 32-bit."""
+
+    def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, key_dim: int,
+                 v_dim: int, conv_taps: int, out_norm_eps: float = 1e-6, prefix: str = "mix"):
+        if num_heads % num_kv_heads:
+            raise ValueError(f"{num_heads} heads are not a multiple of {num_kv_heads} kv heads")
+        if conv_taps < 1:
+            raise ValueError("the convolutions need at least one tap")
+        if key_dim > delta.MAX_KEY_SIZE:
+            raise ValueError(f"a key size of {key_dim} is over the recurrence kernel's "
+                             f"{delta.MAX_KEY_SIZE}")
+        self.hidden_size, self.H, self.G = int(hidden_size), int(num_heads), int(num_kv_heads)
+        self.D, self.Vd, self.taps = int(key_dim), int(v_dim), int(conv_taps)
+        self.eps = float(out_norm_eps)
+        self.prefix = prefix + "." if prefix else ""
+        self.channels = 2 * self.G * self.D + self.H * self.Vd
+        self.conv_off = self.H * self.D * self.Vd            # behind S in a slot
+
+    def _n(self, name):
+        return self.prefix + name
+
+    def tensor_specs(self):
+        H, G, D, Vd, W, t = self.H, self.G, self.D, self.Vd, self.hidden_size, self.taps
+        return [TensorSpec(self._n("q"), (G * D, W)), TensorSpec(self._n("q.conv"), (G * D, t), "f32"),
+                TensorSpec(self._n("k"), (G * D, W)), TensorSpec(self._n("k.conv"), (G * D, t), "f32"),
+                TensorSpec(self._n("v"), (H * Vd, W)),
+                TensorSpec(self._n("v.conv"), (H * Vd, t), "f32"),
+                TensorSpec(self._n("b"), (H, W)), TensorSpec(self._n("a"), (H, W)),
+                TensorSpec(self._n("A_log"), (H,), "f32"),
+                TensorSpec(self._n("dt_bias"), (H,), "f32"),
+                TensorSpec(self._n("norm"), (Vd,), "norm32"),
+                TensorSpec(self._n("g"), (H * Vd, W)), TensorSpec(self._n("o"), (W, H * Vd))]
+
+    def load(self, tensors, dtype, device):
+        def t(name):
+            return tensors[self._n(name)]
+        rows = [t("q"), t("k"), t("v"), t("g"), t("a"), t("b")]
+        self.g_off = self.channels
+        self.a_off = self.g_off + self.H * self.Vd
+        self.b_off = self.a_off + self.H
+        pad = -(self.b_off + self.H) % 8               # rows of the product stay 16-byte aligned
+        if pad:
+            rows.append(torch.zeros((pad, self.hidden_size), dtype=rows[0].dtype, device=device))
+        self.first = ops.Linear(torch.cat(rows, dim=0), None, out_dtype=torch.float32)
+        self.out = ops.Linear(t("o"), None, out_dtype=torch.float32)
+        self.conv_w = torch.cat([t("q.conv"), t("k.conv"), t("v.conv")], dim=0).float().contiguous()
+        self.A_log = t("A_log").float().contiguous()
+        self.dt_bias = t("dt_bias").float().contiguous()
+        self.norm_w = t("norm").float().contiguous()
+
+    def cache_spec(self):
+        return StateSpec((self.conv_off + (self.taps - 1) * self.channels,), torch.float32)
+
+    def forward(self, x, ctx, cache):
+        H, G, D, Vd = self.H, self.G, self.D, self.Vd
+        state = cache.state
+        p = self.first(x)                                    # fp32 [T, q | k | v | g | a | b (| pad)]
+        qn, kn, v, g, beta = delta.prepare_heads(p, self.a_off, self.b_off, self.conv_w,
+                                                 self.dt_bias, self.A_log, state, ctx, H, G, D, Vd,
+                                                 self.taps, self.conv_off)
+        o = delta.recurrence(qn, kn, v, g, beta, state, ctx)
+        y = decay.gated_norm(o.view(-1, H * Vd), p[:, self.g_off:self.g_off + H * Vd], self.norm_w,
+                             Vd, False, self.eps, ctx.dtype)
+        return self.out(y)
+
+
+register_mixer("head_delta", HeadDelta)

@@ -7,6 +7,8 @@ joined at load into one matrix so that one product reads ``y`` once.
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
 from .. import ops
@@ -83,19 +85,21 @@ register_feed_forward("clamped_glu", ClampedGLU)
 
 
 class DenseActivationMLP(FeedForward):
-    """Two matrices with an activation between them: ``W_down act(W_up x + b_up) + b_down`` with
-    ``act = relu^2`` (the only one so far); biases optional.  The output leaves in fp32 for the
-    norm that follows it."""
+    """Two matrices with an activation between them: ``W_down act(W_up x + b_up) + b_down``; biases
+    optional.  ``act`` is ``relu2`` (``relu(z)^2``) or ``xielu``, which has two numbers ``(p, q)`` of
+    its own (the tensor ``act``): ``softplus(p) z^2 + z/2`` above zero and ``(1/2 + softplus(q))
+    (e^z - 1 - z) + z/2`` below.  The output leaves in fp32 for the norm that follows it."""
 
     def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "relu2",
                  bias: bool = True, prefix: str = "mlp", up_name: str = "up",
                  down_name: str = "down"):
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
-        if activation != "relu2":
-            raise ValueError(f"activation {activation!r}: only 'relu2' is there")
+        if activation not in ("relu2", "xielu"):
+            raise ValueError(f"activation {activation!r}: 'relu2' and 'xielu' are there")
         self.activation, self.bias = activation, bool(bias)
         p = prefix + "." if prefix else ""
         self.up_key, self.down_key = p + up_name, p + down_name
+        self.act_key = p + "act" if activation == "xielu" else None
 
     def tensor_specs(self):
         h, i = self.hidden_size, self.intermediate_size
@@ -103,11 +107,19 @@ class DenseActivationMLP(FeedForward):
         if self.bias:
             out += [TensorSpec(self.up_key + ".b", (i,), "bias"),
                     TensorSpec(self.down_key + ".b", (h,), "bias")]
+        if self.act_key:
+            out.append(TensorSpec(self.act_key, (2,), "f32"))
         return out
 
     def load(self, tensors, dtype, device):
         b = (lambda k: tensors[k + ".b"].float().contiguous()) if self.bias else (lambda k: None)
-        self.up = ops.Linear(tensors[self.up_key], b(self.up_key), activation=self.activation)
+        consts = None
+        if self.act_key:
+            p, q = (float(v) for v in tensors[self.act_key].double().cpu())
+            consts = (math.log1p(math.exp(p)) if p < 30 else p,
+                      0.5 + (math.log1p(math.exp(q)) if q < 30 else q))
+        self.up = ops.Linear(tensors[self.up_key], b(self.up_key), activation=self.activation,
+                             act_consts=consts)
         self.down = ops.Linear(tensors[self.down_key], b(self.down_key), out_dtype=torch.float32)
 
     can_defer_bias = True

@@ -81,6 +81,12 @@ class DecoderModel:
         for e in self.plan.run:
             if e.write_cache:
                 out[e.cache] = self.blocks[e.layer].mixer.cache_spec()
+            own = self.blocks[e.layer].state_spec()
+            if (own is None) != (e.block_state is None):
+                raise ValueError(f"a run of layer {e.layer} and its block disagree on whether the "
+                                 "block keeps a state")
+            if own is not None:
+                out[e.block_state] = own
         for e in self.plan.run:
             if not e.write_cache:
                 mine = self.blocks[e.layer].mixer.cache_spec()
@@ -89,9 +95,17 @@ class DecoderModel:
                                      f"{out[e.cache]} but the layer expects {mine}")
         return out
 
+    def _next_input(self, entry, own_state):
+        """What the block before may prepare for ``entry``'s run: nothing where its block's own
+        state is needed for that and not at hand."""
+        if entry.block_state is not None and own_state is None:
+            return None
+        return self.blocks[entry.layer].first_input(own_state)
+
     # ------------------------------------------------------------------ one step
     def forward(self, ctx: StepContext, bind_cache) -> torch.Tensor:
-        """Run the step's tokens; ``bind_cache(run_entry)`` gives the cache binding of a run.
+        """Run the step's tokens; ``bind_cache(run_entry)`` gives the cache binding of a run,
+        ``bind_cache(run_entry, block=True)`` that of its block's own state.
         Returns fp32 logits ``[R, vocab]`` at ``ctx.logit_rows``."""
         delta = None
         x = self.embedding.forward(ctx.token_ids, ctx)
@@ -103,12 +117,19 @@ class DecoderModel:
                 if delta is not None:
                     x, delta = x.float() + delta.float(), None
                 x = self.stream_inputs[e.enter[0]].enter(x, ctx, embedded, e.enter[1])
+            kw = {}
+            if e.block_state is not None:
+                kw["own_state"] = bind_cache(e, block=True)
             if blk.takes_next_norm and i + 1 < len(run) and run[i + 1].enter is None:
                 # the block may prepare the input of the norm that the next run starts with
+                n = run[i + 1]
+                own = None
+                if n.block_state is not None and blk.prepares_shifted_input:
+                    own = bind_cache(n, block=True)
                 x, delta = blk.forward(x, delta, ctx, bind_cache(e),
-                                       then=self.blocks[run[i + 1].layer].first_norm())
+                                       then=self._next_input(n, own), **kw)
             else:
-                x, delta = blk.forward(x, delta, ctx, bind_cache(e))
+                x, delta = blk.forward(x, delta, ctx, bind_cache(e), **kw)
         if ctx.logit_rows.numel() == 0:
             return torch.empty((0, self.plan.vocab_size), dtype=torch.float32, device=ctx.device)
         if isinstance(x, Summed):

@@ -16,14 +16,17 @@ from .base import LazyNorm, Norm, TensorSpec, register_norm
 
 class RMSNorm(Norm):
     """``weight_offset``: the stored weight is an offset from this value (1.0 for weights stored
-    around zero: the norm multiplies by ``1 + w``); the sum is formed once, in 32-bit, at load."""
+    around zero: the norm multiplies by ``1 + w``); the sum is formed once, in 32-bit, at load.
+    ``weight_mult``: a constant the weight is multiplied by, likewise (a factor of what a linear
+    layer behind the norm makes of it, the logits say)."""
 
     def __init__(self, size: int, eps: float, weight_name: str = "weight",
-                 weight_offset: float = 0.0):
+                 weight_offset: float = 0.0, weight_mult: float = 1.0):
         self.size = int(size)
         self.eps = float(eps)
         self.weight_name = weight_name
         self.weight_offset = float(weight_offset)
+        self.weight_mult = float(weight_mult)
         self.weight: torch.Tensor | None = None
         self._w32: torch.Tensor | None = None      # the weight in 32-bit, made when first needed
 
@@ -36,6 +39,8 @@ class RMSNorm(Norm):
         self._w32 = None
         if self.weight_offset:
             self.weight = (self.weight.float() + self.weight_offset).contiguous()
+        if self.weight_mult != 1.0:
+            self.weight = (self.weight.float() * self.weight_mult).contiguous()
 
     def weight32(self) -> torch.Tensor:
         """The weight in 32-bit (made once), for kernels that apply this norm inside a pass of

@@ -40,11 +40,13 @@ class RunEntry:
     ``write_cache=False`` only reads the cache another run has written earlier in the step.
     ``enter = (i, n)``: before this run the stream passes through
     :attr:`ModelPlan.stream_inputs` ``[i]`` as its entry number ``n`` (the start of a pass of a
-    loop, say)."""
+    loop, say).  ``block_state`` names the per-request state of the layer's block itself, beside
+    its mixer's cache (for blocks that keep one)."""
     layer: int
     cache: int
     write_cache: bool = True
     enter: tuple[int, int] | None = None
+    block_state: int | None = None
 
 
 @dataclass(frozen=True)
@@ -75,6 +77,11 @@ class ModelPlan:
                     raise ValueError(f"run[{pos}] and run[{writers[e.cache]}] both write cache "
                                      f"{e.cache}")
                 writers[e.cache] = pos
+            if e.block_state is not None:
+                if e.block_state in writers:
+                    raise ValueError(f"run[{pos}] keeps its block's state as {e.block_state}, "
+                                     f"which run[{writers[e.block_state]}] writes")
+                writers[e.block_state] = pos
         for pos, e in enumerate(self.run):
             if not e.write_cache and (e.cache not in writers or writers[e.cache] > pos):
                 raise ValueError(f"run[{pos}] reads cache {e.cache} before any run writes it")

@@ -10,6 +10,8 @@ in double and rounded to fp32, so host and device cannot disagree on a table ent
 """
 from __future__ import annotations
 
+import math
+
 import numpy as np
 import torch
 
@@ -59,12 +61,22 @@ class PairRotary(PositionEncoding):
     wavelengths: with ``l = 2 pi / f``, ``f`` stays where ``l < original/high``, becomes
     ``f / factor`` where ``l > original/low`` and ``(1 - s) f / factor + s f`` with
     ``s = (original/l - low) / (high - low)`` in between.  ``linear_factor`` divides every
-    frequency (positions stretched evenly).  Nothing is tabulated by position: the
+    frequency (positions stretched evenly).  ``yarn = {factor, original, fast, slow}``: with
+    ``d(t) = dims ln(original / (2 pi t)) / (2 ln base)``, the pairs below ``floor(d(fast))`` keep
+    their frequency, those above ``ceil(d(slow))`` have it divided by ``factor``, a linear ramp
+    over the pair's number lies between, and sine and cosine are multiplied by ``0.1 ln(factor) +
+    1`` (:attr:`mult`).  Nothing is tabulated by position: the
     mixer's kernel forms ``float(p) * f_i`` in 32-bit and takes sine and cosine of it."""
 
     def __init__(self, dims: int, base: float, scaling=None, interleaved: bool = True,
-                 linear_factor: float = 1.0):
+                 linear_factor: float = 1.0, yarn=None):
         self.dims, self.base = int(dims), float(base)
+        self.yarn = None if yarn is None else {k: float(yarn[k]) for k in
+                                               ("factor", "original", "fast", "slow")}
+        if self.yarn is not None and scaling is not None:
+            raise ValueError("frequencies are scaled by 'scaling' or by 'yarn', not both")
+        # what sine and cosine are multiplied by
+        self.mult = 1.0 if self.yarn is None else 0.1 * math.log(self.yarn["factor"]) + 1.0
         self.linear_factor = float(linear_factor)
         if not (self.linear_factor > 0):
             raise ValueError(f"linear_factor must be > 0, got {linear_factor}")
@@ -87,6 +99,15 @@ class PairRotary(PositionEncoding):
             mid = (1.0 - ramp) * f / sc["factor"] + ramp * f
             f = np.where(wave < sc["original"] / sc["high"], f,
                          np.where(wave > sc["original"] / sc["low"], f / sc["factor"], mid))
+        y = self.yarn
+        if y is not None and self.dims:
+            def pair_at(turns):
+                return (self.dims * math.log(y["original"] / (2.0 * math.pi * turns))
+                        / (2.0 * math.log(self.base)))
+            lo = max(math.floor(pair_at(y["fast"])), 0)
+            hi = min(math.ceil(pair_at(y["slow"])), self.dims - 1)
+            ramp = np.clip((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+            f = f / y["factor"] * ramp + f * (1.0 - ramp)
         return (f / self.linear_factor).astype(np.float32)
 
     def load(self, tensors, dtype, device):
