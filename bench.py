@@ -261,7 +261,7 @@ def prefill_timed(eng, tokens: int, reps: int, warmup: int, seed: int):
 
 
 # ----------------------------------------------------------------------------- another design
-# ``--design vilepel|zolapel|pimidra|bapivik``: prefill and decode throughput of another design at layer sizes that
+# ``--design vilepel|zolapel|pimidra|bapivik|lasizen``: prefill and decode throughput of another design at layer sizes that
 # resemble a real model's (random weights), beside Qwen2 at equal width, heads, feed-forward size
 # and layer count.  The default workload and its JSON line are untouched by this option.
 def vilepel_config(width, heads, dim, rot, vdim, rank, window, ff, experts, top, expert_ff,
@@ -359,6 +359,30 @@ def bapivik_config(width, heads, kv_heads, dim, rank, q_rank, window, ff, layers
             "layers": out}
 
 
+def lasizen_config(width, heads, kv_heads, dim, window, ff, layers, vocab=32768):
+    """Windowed attention (rotation, then norms; a sink) and the delta rule with one decay a head in
+    turns, each with a dense xIELU feed-forward."""
+    attention = {"type": "attention", "mixer": {
+        "heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+        "mask": {"size": window},
+        "rot": {"base": 500000.0, "dims": dim // 2,
+                "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    delta = {"type": "delta", "mixer": {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": dim,
+                                        "conv": 4}}
+    return {"architecture": "Lasizen", "width": width, "vocab": vocab, "norm": {"eps": 1e-5},
+            "embedding": {"scale": 1.0}, "logit_scale": 0.5, "torch_dtype": "bfloat16",
+            "layers": [dict((attention, delta)[i % 2], mlp={"kind": "dense", "ff": ff})
+                       for i in range(layers)]}
+
+
+LASIZEN_SIZES = {
+    # width, heads, kv heads, dim, window, two-matrix ff (Vilepel beside it: a three-matrix ff of two
+    # thirds of that)
+    "s": (1024, 8, 2, 64, 512, 4224),
+    "m": (2048, 16, 4, 128, 1024, 8448),
+}
+
+
 BAPIVIK_SIZES = {
     # width, heads, kv heads, dim, latent rank, query rank, window, two-matrix ff (Vilepel beside
     # it: a three-matrix ff of two thirds of that)
@@ -416,6 +440,16 @@ def design_configs(design: str, name: str, layers: int) -> dict:
             "vilepel": vilepel_config(width, heads, dim, dim // 2, dim, rank, window, 2 * ff // 3,
                                       1, 1, 1, layers, routed=False),
         }
+    if design == "lasizen":
+        # beside it the closest design the engine has, Vilepel (attention with a bounded reach and
+        # the delta rule in turns, an fp32 stream), with dense feed-forwards only, at the same width,
+        # heads, head size, window, feed-forward arithmetic and layer count
+        width, heads, kv, dim, window, ff = LASIZEN_SIZES[name]
+        return {
+            "lasizen": lasizen_config(width, heads, kv, dim, window, ff, layers),
+            "vilepel": vilepel_config(width, heads, dim, dim // 2, dim, width // 4, window,
+                                      2 * ff // 3, 1, 1, 1, layers, routed=False),
+        }
     if design == "pimidra":
         # beside it the closest design the engine has, Vilepel (attention with a bounded reach and a
         # recurrent mixer in turns, dense and routed feed-forwards, an fp32 stream), at the same
@@ -444,12 +478,12 @@ def run_design(args) -> int:
     from ginfer_b200.engine.llm import Engine
     out = {"design": args.design,
            "beside": ("vilepel at equal width, heads, head size, feed-forward sizes, reach and "
-                      "layers" if args.design in ("pimidra", "bapivik") else
+                      "layers" if args.design in ("pimidra", "bapivik", "lasizen") else
                       "qwen2 at equal width, heads, feed-forward arithmetic and layer runs"),
            "dtype": "bfloat16", "data": "synthetic", "sizes": {}}
     layers = args.layers or 8
     sizes = {"zolapel": ZOLAPEL_SIZES, "pimidra": PIMIDRA_SIZES,
-             "bapivik": BAPIVIK_SIZES}.get(args.design, DESIGN_SIZES)
+             "bapivik": BAPIVIK_SIZES, "lasizen": LASIZEN_SIZES}.get(args.design, DESIGN_SIZES)
     for name in (args.size.split(",") if args.size else sorted(sizes)):
         cfgs = design_configs(args.design, name, layers)
         width = sizes[name][0]
@@ -477,7 +511,8 @@ def run_design(args) -> int:
 # ----------------------------------------------------------------------------- small workloads
 MICRO = ("gemm_gateup_m8", "gemm_down_m8", "gemm_lmhead_m8", "gemm_gateup_m2048", "gemm_qkv_m2048",
          "attn_decode_b8",
-         "attn_decode_b64", "attn_decode_b1_ctx32768", "prefill_2layers", "bapivik_prefill_4layers")
+         "attn_decode_b64", "attn_decode_b1_ctx32768", "prefill_2layers", "bapivik_prefill_4layers",
+         "lasizen_prefill_2layers")
 
 
 def run_micro(name: str) -> int:
@@ -567,11 +602,12 @@ def run_micro(name: str) -> int:
         torch.cuda.synchronize()
         print(json.dumps({"micro": name, "tokens": PREFILL_TOKENS}))
         return 0
-    if name == "bapivik_prefill_4layers":
-        # one turn of Bapivik's four layers at size m, a 2,048-token prompt three times
+    if name in ("bapivik_prefill_4layers", "lasizen_prefill_2layers"):
+        # one turn of the design's layers at size m, a 2,048-token prompt three times
         from ginfer_b200.engine import StepEntry
         from ginfer_b200.engine.llm import Engine
-        cfg = design_configs("bapivik", "m", 4)["bapivik"]
+        design = name.split("_")[0]
+        cfg = design_configs(design, "m", int(name[-7]))[design]
         eng = Engine(config=cfg, weights_seed=0, dtype="bfloat16", max_num_seqs=4,
                      max_seq_len=CONTEXT, kvcache_block_size=PAGE,
                      num_kvcache_blocks=PREFILL_TOKENS // PAGE + 64, enforce_eager=True)
@@ -796,7 +832,7 @@ def main() -> int:
                     help="tokens a step of the long prompt in --scenario longctx (default 2,048)")
     ap.add_argument("--scenario", choices=SCENARIOS, default=None,
                     help="run a serving workload through the entry point instead of the benchmark")
-    ap.add_argument("--design", choices=["vilepel", "zolapel", "pimidra", "bapivik"], default=None,
+    ap.add_argument("--design", choices=["vilepel", "zolapel", "pimidra", "bapivik", "lasizen"], default=None,
                     help="measure another design beside Qwen2 at equal size instead of the benchmark")
     ap.add_argument("--size", default=None, help="with --design: sizes to run, e.g. s,m")
     args = ap.parse_args()

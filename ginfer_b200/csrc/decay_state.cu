@@ -25,6 +25,7 @@
 //   gated_norm_kernel         a warp a (token, group of channels): RMS norm with a gate, the gate
 //                             before the norm (y = o silu(z), then y / rms(y) w) or behind it
 //                             (o / rms(o) w silu(z)); the weight per channel or shared by the groups.
+//   gated_norm_warp_vec_kernel  the same with four channels an access;
 //   gated_norm_block_kernel   the same with a block a (token, group), for groups over 512 channels;
 //   gated_norm_vec_kernel     with four channels an access and up to 1,024 threads where rows allow.
 //
@@ -382,6 +383,54 @@ __global__ void gated_norm_kernel(const float* __restrict__ o, const G* __restri
 }
 
 
+// The same with four channels an access, the row in registers (NQ quads a lane): groups of up to 128
+// NQ channels, a multiple of four; pointers and row strides aligned to four elements.
+template <typename G, typename T, int NQ>
+__global__ void gated_norm_warp_vec_kernel(const float* __restrict__ o, const G* __restrict__ gate,
+                                           int gate_ld, const float* __restrict__ w, int w_shared,
+                                           int gate_mode, float eps, T* __restrict__ out, int units,
+                                           int groups, int gs) {
+  const int unit = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int sig = gate_mode >> 1, gate_first = gate_mode & 1;
+  pdl_trigger();
+  pdl_wait();
+  if (unit >= units) return;
+  const int r = unit / groups, gi = unit - r * groups, nq = gs >> 2;
+  const float* orow = o + (size_t)r * groups * gs + (size_t)gi * gs;
+  const G* grow = gate + (size_t)r * gate_ld + (size_t)gi * gs;
+  const float* wrow = w + (w_shared ? 0 : (size_t)gi * gs);
+  T* dst = out + (size_t)r * groups * gs + (size_t)gi * gs;
+  float y[NQ][4], z[NQ][4];
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < NQ; ++u) {
+    const int q = lane + 32 * u;
+    if (q < nq) {
+      Quad<float>::load(orow + 4 * q, y[u]);
+      Quad<G>::load(grow + 4 * q, z[u]);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        z[u][i] = ds_gate(z[u][i], sig);
+        if (gate_first) y[u][i] *= z[u][i];
+        ss = fmaf(y[u][i], y[u][i], ss);
+      }
+    }
+  }
+  ss = warp_sum(ss);
+  const float inv = 1.f / sqrtf(ss / (float)gs + eps);
+#pragma unroll
+  for (int u = 0; u < NQ; ++u) {
+    const int q = lane + 32 * u;
+    if (q < nq) {
+      float wq[4];
+      Quad<float>::load(wrow + 4 * q, wq);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) y[u][i] *= gate_first ? inv * wq[i] : inv * wq[i] * z[u][i];
+      Quad<T>::store(dst + 4 * q, y[u]);
+    }
+  }
+}
+
 // The same with a block a unit, for groups of thousands of channels (a warp would walk them alone).
 template <typename G, typename T>
 __global__ void __launch_bounds__(256)
@@ -601,8 +650,9 @@ GF_EXPORT int gf_gated_norm(const float* o, const void* gate, int gate_ld, int g
   const dim3 grid((units + 3) / 4), block(128);
   const bool wide = gs > kGatedNormWarpMax;
   auto quads = [](const void* p, size_t elem) { return ((uintptr_t)p % (4 * elem)) == 0; };
-  const bool vec = wide && gs % 4 == 0 && gate_ld % 4 == 0 && quads(o, 4) && quads(w, 4) &&
+  const bool quad_rows = gs % 4 == 0 && gate_ld % 4 == 0 && quads(o, 4) && quads(w, 4) &&
                    quads(gate, gate_dtype == GF_F32 ? 4 : 2) && quads(out, dtype == GF_F32 ? 4 : 2);
+  const bool vec = wide && quad_rows;
   const int vthreads = gs / 4 >= 1024 ? 1024 : (gs / 4 + 31) / 32 * 32;
 #define GF_GO(GT, OT)                                                                              \
   {                                                                                                \
@@ -610,6 +660,14 @@ GF_EXPORT int gf_gated_norm(const float* o, const void* gate, int gate_ld, int g
       return launch_kernel(gated_norm_vec_kernel<GT, OT>, dim3(units), dim3(vthreads), 0, st, o,   \
                            (const GT*)gate, gate_ld, w, w_shared, gate_first, eps, (OT*)out,       \
                            groups, gs);                                                            \
+    if (!wide && quad_rows && gs <= 128)                                                           \
+      return launch_kernel(gated_norm_warp_vec_kernel<GT, OT, 1>, grid, block, 0, st, o,           \
+                           (const GT*)gate, gate_ld, w, w_shared, gate_first, eps, (OT*)out,       \
+                           units, groups, gs);                                                     \
+    if (!wide && quad_rows)                                                                        \
+      return launch_kernel(gated_norm_warp_vec_kernel<GT, OT, 4>, grid, block, 0, st, o,           \
+                           (const GT*)gate, gate_ld, w, w_shared, gate_first, eps, (OT*)out,       \
+                           units, groups, gs);                                                     \
     if (wide)                                                                                      \
       return launch_kernel(gated_norm_block_kernel<GT, OT>, dim3(units), dim3(256), 0, st, o,      \
                            (const GT*)gate, gate_ld, w, w_shared, gate_first, eps, (OT*)out,       \

@@ -16,6 +16,8 @@
 //                            independent: four lanes or a warp share a column (a share of the rows
 //                            each, in registers).  The tokens' operands come through two stages of
 //                            shared memory, a chunk ahead (cp.async).
+//   delta_chunk_coef_kernel, delta_chunk_recurrence_kernel   the recurrence of long portions with one
+//                            decay a head, eight tokens at a time (see there).
 //   delta_output_kernel      a warp a (token, head): o / rms(o) * w * sigmoid(gate).
 #include "common.cuh"
 
@@ -437,6 +439,273 @@ delta_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ 
   }
 }
 
+// ---- eight tokens at a time ---------------------------------------------------------------------
+// With one decay a head the recurrence over a chunk of tokens 0 .. 7 that starts from S needs S only
+// in products that do not wait for one another.  With G_i = g_0 .. g_i, R(j, i) = g_(j+1) .. g_i:
+//
+//   u_i = beta_i (v_i - G_i S^T k_i) - sum_(j<i) L_ij u_j,   L_ij = beta_i R(j, i) k_j.k_i
+//   o_i = G_i S^T q_i + sum_(j<=i) M_ij u_j,                 M_ij = R(j, i) k_j.q_i
+//   S  <- G_7 S + sum_j R(j, 7) k_j u_j^T
+//
+// (ratios of decays are products of the factors between the two tokens, never quotients).  The chain
+// from token to token is then eight multiply-adds in registers a chunk, instead of a pass over S and a
+// reduction across lanes a token.  Everything is 32-bit multiply-adds.
+constexpr int CT = 8;                                          // tokens a chunk
+constexpr int kCoefL = 0, kCoefM = 64, kCoefG = 128, kCoefE = 136, kCoefBeta = 144, kCoefs = 152;
+
+// Chunks of request b start at the packed number cu[b] / CT + b; no two requests' chunks meet.
+__device__ __forceinline__ int chunk_number(int first_row, int b, int c) { return first_row / CT + b + c; }
+
+// A warp a (chunk, kv head): the 64 dot products k_j.k_i (j < i) and k_j.q_i (j <= i), then for every
+// head of the group L, M, G, E (E_j = R(j, 7)) and beta.  Tokens behind the portion's end count as
+// k = q = 0, g = 1, beta = 0.
+__global__ void __launch_bounds__(128)
+delta_chunk_coef_kernel(const float* __restrict__ qn, const float* __restrict__ kn,
+                        const float* __restrict__ g, const float* __restrict__ beta,
+                        const int* __restrict__ cu_seqlens, DeltaDims dm, float* __restrict__ coef) {
+  const int lane = threadIdx.x & 31;
+  const int c = blockIdx.x * 4 + (threadIdx.x >> 5), b = blockIdx.y, kvh = blockIdx.z;
+  pdl_wait();
+  const int t0 = cu_seqlens[b], ta = t0 + c * CT, n = min(CT, cu_seqlens[b + 1] - ta);
+  if (n <= 0) return;
+  const int D = dm.D, H = dm.H, per = H / dm.G;
+  const size_t GD = (size_t)dm.G * D;
+  // pair (a, e) = (m / 8, m % 8): k_e.k_a for a > e, k_a.q_e for a <= e
+  float val[64];
+#pragma unroll
+  for (int m = 0; m < 64; ++m) val[m] = 0.f;
+  for (int d = 4 * lane; d < D; d += 128) {
+    float k[CT][4], q[CT][4];
+#pragma unroll
+    for (int i = 0; i < CT; ++i) {
+#pragma unroll
+      for (int x = 0; x < 4; ++x) k[i][x] = q[i][x] = 0.f;
+      if (i < n) {
+        const size_t at = (size_t)(ta + i) * GD + (size_t)kvh * D + d;
+        Quad<float>::load(kn + at, k[i]);
+        Quad<float>::load(qn + at, q[i]);
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < 64; ++m) {
+      const int a = m >> 3, e = m & 7;
+#pragma unroll
+      for (int x = 0; x < 4; ++x) val[m] = fmaf(k[a > e ? e : a][x], a > e ? k[a][x] : q[e][x], val[m]);
+    }
+  }
+  // add up across the lanes, halving the values each lane carries: lane l ends with m = l, l + 32
+#pragma unroll
+  for (int half = 16; half >= 1; half >>= 1) {
+    const bool up = lane & half;
+    // values that differ in this bit of m are neighbours at distance `half`; what is left of the
+    // list is indexed by m with the higher bits already fixed to the lane's
+#pragma unroll
+    for (int hi = 0; hi < 2; ++hi)
+#pragma unroll
+      for (int m = 0; m < half; ++m) {
+        const float lo_v = val[32 * hi + m], hi_v = val[32 * hi + m + half];
+        const float got = __shfl_xor_sync(0xffffffffu, up ? lo_v : hi_v, half);
+        val[32 * hi + m] = (up ? hi_v : lo_v) + got;
+      }
+  }
+  const float mine[2] = {val[0], val[32]};
+  float* base = coef + ((size_t)chunk_number(t0, b, c) * H + (size_t)kvh * per) * kCoefs;
+  for (int hh = 0; hh < per; ++hh) {
+    const int h = kvh * per + hh;
+    const bool real = lane < n;
+    const float gl = real ? g[(size_t)(ta + lane) * H + h] : 1.f;
+    const float bl = real ? beta[(size_t)(ta + lane) * H + h] : 0.f;
+    float* dst = base + (size_t)hh * kCoefs;
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int m = lane + 32 * x, a = m >> 3, e = m & 7;
+      const int i = a > e ? a : e, j = a > e ? e : a;          // j <= i
+      float r = 1.f;
+#pragma unroll
+      for (int s = 1; s < CT; ++s) {
+        const float gs = __shfl_sync(0xffffffffu, gl, s);
+        if (s > j && s <= i) r *= gs;
+      }
+      const float bi = __shfl_sync(0xffffffffu, bl, i);
+      if (a > e) {
+        dst[kCoefL + i * CT + j] = bi * r * mine[x];
+        dst[kCoefM + j * CT + i] = 0.f;                         // (M is read as whole rows)
+      } else {
+        dst[kCoefM + i * CT + j] = r * mine[x];
+        if (i == j) dst[kCoefL + i * CT + j] = 0.f;
+      }
+    }
+    float G = 1.f, E = 1.f;
+#pragma unroll
+    for (int s = 0; s < CT; ++s) {
+      const float gs = __shfl_sync(0xffffffffu, gl, s);
+      if (s <= lane) G *= gs;
+      if (s > lane) E *= gs;
+    }
+    if (lane < CT) {
+      dst[kCoefG + lane] = G;
+      dst[kCoefE + lane] = E;
+      dst[kCoefBeta + lane] = bl;
+    }
+  }
+}
+
+// A block = (request, head, 16 columns of S); eight lanes a column.  Lane p of a column owns the rows
+// 4 (p + 8 i) .. + 3, i < DPER / 4, so that the lanes' reads of a token's k and q are one run of
+// shared memory.  Stages as in the kernel above, one barrier a chunk.
+template <int DPER>
+__global__ void __launch_bounds__(128)
+delta_chunk_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ kn,
+                              const float* __restrict__ v, const float* __restrict__ coef,
+                              float* __restrict__ state, const int* __restrict__ cu_seqlens,
+                              const int* __restrict__ slot_ids, DeltaDims dm, float* __restrict__ o) {
+  constexpr int LANES = 8, Dp = LANES * DPER, COLS = 128 / LANES, NQ = DPER / 4;
+  constexpr int kQ = CT * Dp, kVc = 2 * CT * Dp, kC = kVc + CT * COLS, kStage = kC + kCoefs;
+  extern __shared__ __align__(16) float stage[];               // [kStages][kStage]
+  const int b = blockIdx.x / dm.H, h = blockIdx.x - b * dm.H;
+  const int p = threadIdx.x % LANES, lc = threadIdx.x / LANES;
+  const int col0 = blockIdx.y * COLS, col = col0 + lc;
+  pdl_trigger();
+  const int D = dm.D, Vd = dm.Vd;
+  for (int i = threadIdx.x; i < kStages * kStage; i += blockDim.x) stage[i] = 0.f;
+  __syncthreads();
+  pdl_wait();
+  const bool col_ok = col < Vd;
+  const int cj = col_ok ? col : 0;
+  const int kvh = h / (dm.H / dm.G);
+  float* Sg = state + (size_t)slot_ids[b] * dm.state_stride + ((size_t)h * D) * Vd + cj;
+  float S[NQ][4];
+#pragma unroll
+  for (int i = 0; i < NQ; ++i)
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      const int row = 4 * (p + LANES * i) + x;
+      S[i][x] = row < D ? Sg[(size_t)row * Vd] : 0.f;
+    }
+  const int t0 = cu_seqlens[b], t1 = cu_seqlens[b + 1];
+  const size_t GD = (size_t)dm.G * D, HV = (size_t)dm.H * Vd;
+  const int vq = min(COLS, Vd - col0) >> 2, dq = D >> 2;
+  const int nchunks = (t1 - t0 + CT - 1) / CT;
+  const float* coef0 = coef + ((size_t)chunk_number(t0, b, 0) * dm.H + h) * kCoefs;
+  auto copy16 = [](float* dst, const float* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+  };
+  auto ask = [&](int c) {
+    float* st = stage + (size_t)(c % kStages) * kStage;
+    const int ta = t0 + c * CT, n = min(CT, t1 - ta);
+    for (int e = threadIdx.x; e < n * dq; e += blockDim.x) {
+      const int t = e / dq, d = 4 * (e - t * dq);
+      const size_t at = (size_t)(ta + t) * GD + (size_t)kvh * D + d;
+      copy16(st + t * Dp + d, kn + at);
+      copy16(st + kQ + t * Dp + d, qn + at);
+    }
+    for (int e = threadIdx.x; e < n * vq; e += blockDim.x) {
+      const int t = e / vq, d = 4 * (e - t * vq);
+      copy16(st + kVc + t * COLS + d, v + (size_t)(ta + t) * HV + (size_t)h * Vd + col0 + d);
+    }
+    for (int e = threadIdx.x; e < kCoefs / 4; e += blockDim.x)
+      copy16(st + kC + 4 * e, coef0 + (size_t)c * dm.H * kCoefs + 4 * e);
+  };
+  for (int c = 0; c < kStages - 1; ++c) {
+    if (c < nchunks) ask(c);
+    copy_async_commit();
+  }
+  for (int c = 0; c < nchunks; ++c) {
+    copy_async_wait<kStages - 2>();
+    __syncthreads();                 // chunk c has landed for all, and all have left chunk c - 1
+    if (c + kStages - 1 < nchunks) ask(c + kStages - 1);       // into the stage of chunk c - 1
+    copy_async_commit();
+    const float* st = stage + (size_t)(c % kStages) * kStage;
+    const float* cf = st + kC;
+    // this lane's share of S^T k_i (x[i]) and S^T q_i (x[8 + i])
+    float x[2 * CT];
+#pragma unroll
+    for (int i = 0; i < 2 * CT; ++i) x[i] = 0.f;
+#pragma unroll
+    for (int i = 0; i < NQ; ++i) {
+      const float* at = st + 4 * (p + LANES * i);
+#pragma unroll
+      for (int t = 0; t < 2 * CT; ++t) {
+        const float4 a = *reinterpret_cast<const float4*>(at + t * Dp);
+        x[t] = fmaf(S[i][0], a.x, fmaf(S[i][1], a.y, fmaf(S[i][2], a.z, fmaf(S[i][3], a.w, x[t]))));
+      }
+    }
+    // add up across the column's lanes; lane p ends with the sums of token p
+#pragma unroll
+    for (int half = CT / 2; half >= 1; half >>= 1) {
+      const bool up = p & half;
+#pragma unroll
+      for (int hi = 0; hi < 2; ++hi)
+#pragma unroll
+        for (int m = 0; m < half; ++m) {
+          const float lo_v = x[CT * hi + m], hi_v = x[CT * hi + m + half];
+          const float got = __shfl_xor_sync(0xffffffffu, up ? lo_v : hi_v, half);
+          x[CT * hi + m] = (up ? hi_v : lo_v) + got;
+        }
+    }
+    const float Gp = cf[kCoefG + p];
+    const float rp = cf[kCoefBeta + p] * (st[kVc + p * COLS + lc] - Gp * x[0]);
+    float u[CT];
+#pragma unroll
+    for (int i = 0; i < CT; ++i) u[i] = __shfl_sync(0xffffffffu, rp, i, LANES);
+#pragma unroll
+    for (int j = 0; j < CT - 1; ++j)
+#pragma unroll
+      for (int i = j + 1; i < CT; ++i) u[i] = fmaf(-cf[kCoefL + i * CT + j], u[j], u[i]);
+    {
+      const float4* Mp = reinterpret_cast<const float4*>(cf + kCoefM + p * CT);
+      const float4 m0 = Mp[0], m1 = Mp[1];
+      float out = Gp * x[CT];
+      out = fmaf(m0.x, u[0], fmaf(m0.y, u[1], fmaf(m0.z, u[2], fmaf(m0.w, u[3], out))));
+      out = fmaf(m1.x, u[4], fmaf(m1.y, u[5], fmaf(m1.z, u[6], fmaf(m1.w, u[7], out))));
+      const int row = t0 + c * CT + p;
+      if (col_ok && row < t1) o[(size_t)row * HV + (size_t)h * Vd + col] = out;
+    }
+    if (DPER > 16) asm volatile("" ::: "memory");   // read k again: there are no registers to keep it
+    const float Gc = cf[kCoefG + CT - 1];
+#pragma unroll
+    for (int j = 0; j < CT; ++j) u[j] *= cf[kCoefE + j];
+#pragma unroll
+    for (int i = 0; i < NQ; ++i) {
+      const float* at = st + 4 * (p + LANES * i);
+#pragma unroll
+      for (int y = 0; y < 4; ++y) S[i][y] *= Gc;
+#pragma unroll
+      for (int t = 0; t < CT; ++t) {
+        const float4 a = *reinterpret_cast<const float4*>(at + t * Dp);
+        S[i][0] = fmaf(a.x, u[t], S[i][0]);
+        S[i][1] = fmaf(a.y, u[t], S[i][1]);
+        S[i][2] = fmaf(a.z, u[t], S[i][2]);
+        S[i][3] = fmaf(a.w, u[t], S[i][3]);
+      }
+    }
+  }
+  if (col_ok) {
+#pragma unroll
+    for (int i = 0; i < NQ; ++i)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int row = 4 * (p + LANES * i) + x;
+        if (row < D) Sg[(size_t)row * Vd] = S[i][x];
+      }
+  }
+}
+
+template <int DPER>
+static int launch_chunks(const float* qn, const float* kn, const float* v, const float* coef,
+                         float* state, const int* cu_seqlens, const int* slot_ids, int B,
+                         const DeltaDims& dm, float* o, cudaStream_t st) {
+  const size_t smem = (size_t)kStages * (2 * CT * 8 * DPER + CT * 16 + kCoefs) * sizeof(float);
+  static OncePerDevice attrs;
+  if (int rc = attrs.run([&] {
+        return cudaFuncSetAttribute(delta_chunk_recurrence_kernel<DPER>,
+                                    cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      }))
+    return rc;
+  return launch_kernel(delta_chunk_recurrence_kernel<DPER>, dim3(B * dm.H, (dm.Vd + 15) / 16),
+                       dim3(128), smem, st, qn, kn, v, coef, state, cu_seqlens, slot_ids, dm, o);
+}
+
 template <typename T>
 __global__ void delta_output_kernel(const float* __restrict__ o, const T* __restrict__ gate,
                                     int gate_ld, const float* __restrict__ w, float eps,
@@ -548,15 +817,34 @@ GF_EXPORT int gf_delta_prepare_heads(const float* proj, int ld, int a_off, int b
                        0, st, proj, ld, state, cu_seqlens, slot_ids, dm);
 }
 
-// one_decay: g is [T, H] (a decay a head), else [T, H, D].
+// fp32 words of scratch with which gf_delta_recurrence takes eight tokens at a time (one decay a head).
+GF_EXPORT long long gf_delta_chunk_words(int T, int B, int H) {
+  return (long long)(T / CT + B + 1) * H * kCoefs;
+}
+
+// one_decay: g is [T, H] (a decay a head), else [T, H, D].  scratch (gf_delta_chunk_words; null: token
+// by token) and max_q_len, the longest portion, are for steps with one decay a head.
 GF_EXPORT int gf_delta_recurrence(const float* qn, const float* kn, const float* v, const float* g,
                                   const float* beta, float* state, const int* cu_seqlens,
                                   const int* slot_ids, int B, int H, int G, int D, int Vd,
-                                  int state_stride, float* o, int one_decay, void* stream) {
+                                  int state_stride, float* o, int one_decay, float* scratch,
+                                  int max_q_len, void* stream) {
   if (B <= 0) return 0;
   if (H % G) return -3;
   const DeltaDims dm = dims_of(H, G, D, Vd, 1, state_stride, 0);
   auto st = (cudaStream_t)stream;
+  if (one_decay && scratch && D % 4 == 0 && Vd % 4 == 0 && D <= 256 && B <= 65535 && G <= 65535 &&
+      (((uintptr_t)qn | (uintptr_t)kn | (uintptr_t)v | (uintptr_t)scratch) & 15) == 0) {
+    const int chunks = (max_q_len + CT - 1) / CT;
+    if (int rc = launch_kernel(delta_chunk_coef_kernel, dim3((chunks + 3) / 4, B, G), dim3(128), 0, st,
+                               qn, kn, g, beta, cu_seqlens, dm, scratch))
+      return rc;
+    if (D <= 32) return launch_chunks<4>(qn, kn, v, scratch, state, cu_seqlens, slot_ids, B, dm, o, st);
+    if (D <= 64) return launch_chunks<8>(qn, kn, v, scratch, state, cu_seqlens, slot_ids, B, dm, o, st);
+    if (D <= 128)
+      return launch_chunks<16>(qn, kn, v, scratch, state, cu_seqlens, slot_ids, B, dm, o, st);
+    return launch_chunks<32>(qn, kn, v, scratch, state, cu_seqlens, slot_ids, B, dm, o, st);
+  }
   // few (request, head, column) triples: a warp (sixteen lanes for key sizes up to 64) a column
   // instead of four lanes (see the kernel)
   const bool wide = (long long)B * H * ((Vd + 31) / 32) < 2 * 148;

@@ -10,6 +10,9 @@ from . import _code, _cuda, _fn, _ok, _p, _stream
 
 
 MAX_KEY_SIZE = 256        # the recurrence kernel's largest
+# Steps with a portion of at least this many tokens take the recurrence with one decay a head eight
+# tokens at a time.
+CHUNKED_MIN_TOKENS = 16
 
 
 def prepare(proj: torch.Tensor, b_off: int, a: torch.Tensor, conv_w: torch.Tensor,
@@ -81,17 +84,31 @@ def prepare_heads(proj: torch.Tensor, a_off: int, b_off: int, conv_w: torch.Tens
     return qn, kn, v, g, beta
 
 
+def _fn_words():
+    from ctypes import c_longlong
+
+    from .build import load_library
+    f = load_library("delta_rule").gf_delta_chunk_words
+    f.argtypes, f.restype = [c_int] * 3, c_longlong
+    return f
+
+
 def recurrence(qn, kn, v, g, beta, state: torch.Tensor, ctx) -> torch.Tensor:
     """Advance every request's state over its tokens of this step; returns ``o [T, H, Vd]`` fp32.
-    ``g``: ``[T, H, D]``, or ``[T, H]`` for one decay a head."""
+    ``g``: ``[T, H, D]``, or ``[T, H]`` for one decay a head (long portions then go eight tokens at a
+    time)."""
     T, G, D = qn.shape
     H, Vd = v.shape[1], v.shape[2]
     o = torch.empty((T, H, Vd), dtype=torch.float32, device=qn.device)
     f = _fn("delta_rule", "gf_delta_recurrence",
-            [c_void_p] * 8 + [c_int] * 6 + [c_void_p, c_int, c_void_p])
+            [c_void_p] * 8 + [c_int] * 6 + [c_void_p, c_int, c_void_p, c_int, c_void_p])
+    scratch, longest = None, int(ctx.max_q_len) if g.dim() == 2 else 0
+    if longest >= CHUNKED_MIN_TOKENS:
+        words = _fn_words()(T, ctx.num_seqs, H)
+        scratch = torch.empty(words, dtype=torch.float32, device=qn.device)
     rc = f(_p(qn), _p(kn), _p(v), _p(g), _p(beta), _p(state), _p(ctx.cu_seqlens_q),
            _p(ctx.slot_ids), ctx.num_seqs, H, G, D, Vd, state.stride(0), _p(o), int(g.dim() == 2),
-           _stream())
+           _p(scratch), longest, _stream())
     if rc == -3:
         raise ValueError(f"the delta-rule recurrence takes key sizes up to {MAX_KEY_SIZE}, got {D}")
     _ok(rc, "delta_recurrence")

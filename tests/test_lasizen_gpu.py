@@ -719,6 +719,57 @@ def test_delta_rule_with_one_decay_a_head(G, H, D, Vd, taps):
         assert float((state[[1, 3]] - 5.0).abs().max()) == 0.0
 
 
+@pytest.mark.parametrize("D, Vd, per", [(16, 24, 1), (20, 8, 3), (64, 40, 2), (128, 128, 1), (200, 12, 2)])
+def test_eight_tokens_at_a_time_agree_with_one_by_one(D, Vd, per):
+    """The recurrence of long portions against the token-by-token kernel and the plain one, from a
+    state that is not zero, over portions of 16 to 100 tokens beside single ones (ends inside a
+    chunk); keys that repeat with a step size of one (every token undoes the last one's write),
+    decays of exactly one and decays that forget at once."""
+    from ginfer_b200.ops import delta
+    g0 = torch.Generator().manual_seed(D)
+    G, H = 2, 2 * per
+    q_lens, slots = [100, 1, 16, 23, 40], [3, 0, 5, 1, 2]
+    T = sum(q_lens)
+    k = plain.unit(torch.randn(T, G, D, generator=g0))
+    k[101:117, 0] = k[101, 0]                               # one key for a whole portion
+    q = plain.unit(torch.randn(T, G, D, generator=g0)) * D ** -0.5
+    v = torch.randn(T, H, Vd, generator=g0)
+    beta = torch.rand(T, H, generator=g0)
+    beta[101:117] = 1.0
+    gg = torch.rand(T, H, generator=g0) ** 0.2
+    gg[0:40, 0] = 1.0
+    gg[50::7, -1] = 1e-30
+    S0 = torch.randn(6, H * D * Vd, generator=g0)
+    args = [t.float().cuda().contiguous() for t in (q, k, v, gg, beta)]
+    ctx = packed(q_lens, slots)
+    outs = []
+    for min_tokens in (16, 1 << 30):
+        old, delta.CHUNKED_MIN_TOKENS = delta.CHUNKED_MIN_TOKENS, min_tokens
+        try:
+            state = S0.cuda()
+            outs.append((delta.recurrence(*args, state, ctx).cpu(), state.cpu()))
+        finally:
+            delta.CHUNKED_MIN_TOKENS = old
+    (o8, s8), (o1, s1) = outs
+    scale = float(o1.abs().max())
+    assert float((o8 - o1).abs().max()) <= 2e-5 * scale and not torch.equal(o8, o1)
+    assert float((s8 - s1).abs().max()) <= 2e-5 * float(s1.abs().max())
+    assert torch.equal(s8[4], S0[4])
+    at = 0
+    for n, slot in zip(q_lens, slots):
+        S = S0[slot].double().view(H, D, Vd).clone()
+        for t in range(at, at + n):
+            for h in range(H):
+                kk, qq = k[t, h // per].double(), q[t, h // per].double()
+                S[h] = float(gg[t, h]) * S[h]
+                u = float(beta[t, h]) * (v[t, h].double() - S[h].T @ kk)
+                S[h] = S[h] + torch.outer(kk, u)
+                want = S[h].T @ qq
+                assert float((o8[t, h].double() - want).abs().max()) <= 5e-5 * scale, (t, h)
+        assert float((s8[slot].double() - S.view(-1)).abs().max()) <= 5e-5 * float(S.abs().max())
+        at += n
+
+
 def test_delta_operands_of_a_long_prompt_among_others():
     """Enough tokens that a warp walks over runs of them: runs that start inside a portion, at its
     start, and that cross from one request to the next."""
