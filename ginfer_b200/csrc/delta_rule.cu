@@ -550,16 +550,16 @@ delta_chunk_coef_kernel(const float* __restrict__ qn, const float* __restrict__ 
   }
 }
 
-// A block = (request, head, 16 columns of S); eight lanes a column.  Lane p of a column owns the rows
-// 4 (p + 8 i) .. + 3, i < DPER / 4, so that the lanes' reads of a token's k and q are one run of
+// A block = (request, head, 16 columns of S); LANES (8 or 16) lanes a column.  Lane p of a column owns
+// the rows 4 (p + LANES i) .. + 3, i < DPER / 4, so that the lanes' reads of a token's k and q are one run of
 // shared memory.  Stages as in the kernel above, one barrier a chunk.
-template <int DPER>
-__global__ void __launch_bounds__(128)
+template <int DPER, int LANES>
+__global__ void __launch_bounds__(16 * LANES)
 delta_chunk_recurrence_kernel(const float* __restrict__ qn, const float* __restrict__ kn,
                               const float* __restrict__ v, const float* __restrict__ coef,
                               float* __restrict__ state, const int* __restrict__ cu_seqlens,
                               const int* __restrict__ slot_ids, DeltaDims dm, float* __restrict__ o) {
-  constexpr int LANES = 8, Dp = LANES * DPER, COLS = 128 / LANES, NQ = DPER / 4;
+  constexpr int Dp = LANES * DPER, COLS = 16, NQ = DPER / 4;
   constexpr int kQ = CT * Dp, kVc = 2 * CT * Dp, kC = kVc + CT * COLS, kStage = kC + kCoefs;
   extern __shared__ __align__(16) float stage[];               // [kStages][kStage]
   const int b = blockIdx.x / dm.H, h = blockIdx.x - b * dm.H;
@@ -630,21 +630,23 @@ delta_chunk_recurrence_kernel(const float* __restrict__ qn, const float* __restr
         x[t] = fmaf(S[i][0], a.x, fmaf(S[i][1], a.y, fmaf(S[i][2], a.z, fmaf(S[i][3], a.w, x[t]))));
       }
     }
-    // add up across the column's lanes; lane p ends with the sums of token p
+    // add up across the column's lanes: of eight, lane p ends with both sums of token p; of sixteen,
+    // lane p with S^T k of token p or S^T q of token p - 8
 #pragma unroll
-    for (int half = CT / 2; half >= 1; half >>= 1) {
+    for (int half = LANES / 2; half >= 1; half >>= 1) {
       const bool up = p & half;
 #pragma unroll
-      for (int hi = 0; hi < 2; ++hi)
+      for (int hi = 0; hi < 2 * CT / LANES; ++hi)
 #pragma unroll
         for (int m = 0; m < half; ++m) {
-          const float lo_v = x[CT * hi + m], hi_v = x[CT * hi + m + half];
+          const float lo_v = x[LANES * hi + m], hi_v = x[LANES * hi + m + half];
           const float got = __shfl_xor_sync(0xffffffffu, up ? lo_v : hi_v, half);
-          x[CT * hi + m] = (up ? hi_v : lo_v) + got;
+          x[LANES * hi + m] = (up ? hi_v : lo_v) + got;
         }
     }
-    const float Gp = cf[kCoefG + p];
-    const float rp = cf[kCoefBeta + p] * (st[kVc + p * COLS + lc] - Gp * x[0]);
+    const int tok = p % CT;                                     // the token this lane looks after
+    const float Gp = cf[kCoefG + tok];
+    const float rp = cf[kCoefBeta + tok] * (st[kVc + tok * COLS + lc] - Gp * x[0]);
     float u[CT];
 #pragma unroll
     for (int i = 0; i < CT; ++i) u[i] = __shfl_sync(0xffffffffu, rp, i, LANES);
@@ -653,15 +655,14 @@ delta_chunk_recurrence_kernel(const float* __restrict__ qn, const float* __restr
 #pragma unroll
       for (int i = j + 1; i < CT; ++i) u[i] = fmaf(-cf[kCoefL + i * CT + j], u[j], u[i]);
     {
-      const float4* Mp = reinterpret_cast<const float4*>(cf + kCoefM + p * CT);
+      const float4* Mp = reinterpret_cast<const float4*>(cf + kCoefM + tok * CT);
       const float4 m0 = Mp[0], m1 = Mp[1];
-      float out = Gp * x[CT];
+      float out = Gp * (LANES == CT ? x[CT] : x[0]);
       out = fmaf(m0.x, u[0], fmaf(m0.y, u[1], fmaf(m0.z, u[2], fmaf(m0.w, u[3], out))));
       out = fmaf(m1.x, u[4], fmaf(m1.y, u[5], fmaf(m1.z, u[6], fmaf(m1.w, u[7], out))));
-      const int row = t0 + c * CT + p;
-      if (col_ok && row < t1) o[(size_t)row * HV + (size_t)h * Vd + col] = out;
+      const int row = t0 + c * CT + tok;
+      if (col_ok && row < t1 && p >= LANES - CT) o[(size_t)row * HV + (size_t)h * Vd + col] = out;
     }
-    if (DPER > 16) asm volatile("" ::: "memory");   // read k again: there are no registers to keep it
     const float Gc = cf[kCoefG + CT - 1];
 #pragma unroll
     for (int j = 0; j < CT; ++j) u[j] *= cf[kCoefE + j];
@@ -691,19 +692,19 @@ delta_chunk_recurrence_kernel(const float* __restrict__ qn, const float* __restr
   }
 }
 
-template <int DPER>
+template <int DPER, int LANES>
 static int launch_chunks(const float* qn, const float* kn, const float* v, const float* coef,
                          float* state, const int* cu_seqlens, const int* slot_ids, int B,
                          const DeltaDims& dm, float* o, cudaStream_t st) {
-  const size_t smem = (size_t)kStages * (2 * CT * 8 * DPER + CT * 16 + kCoefs) * sizeof(float);
+  const size_t smem = (size_t)kStages * (2 * CT * LANES * DPER + CT * 16 + kCoefs) * sizeof(float);
   static OncePerDevice attrs;
   if (int rc = attrs.run([&] {
-        return cudaFuncSetAttribute(delta_chunk_recurrence_kernel<DPER>,
+        return cudaFuncSetAttribute(delta_chunk_recurrence_kernel<DPER, LANES>,
                                     cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       }))
     return rc;
-  return launch_kernel(delta_chunk_recurrence_kernel<DPER>, dim3(B * dm.H, (dm.Vd + 15) / 16),
-                       dim3(128), smem, st, qn, kn, v, coef, state, cu_seqlens, slot_ids, dm, o);
+  return launch_kernel(delta_chunk_recurrence_kernel<DPER, LANES>, dim3(B * dm.H, (dm.Vd + 15) / 16),
+                       dim3(16 * LANES), smem, st, qn, kn, v, coef, state, cu_seqlens, slot_ids, dm, o);
 }
 
 template <typename T>
@@ -839,11 +840,14 @@ GF_EXPORT int gf_delta_recurrence(const float* qn, const float* kn, const float*
     if (int rc = launch_kernel(delta_chunk_coef_kernel, dim3((chunks + 3) / 4, B, G), dim3(128), 0, st,
                                qn, kn, g, beta, cu_seqlens, dm, scratch))
       return rc;
-    if (D <= 32) return launch_chunks<4>(qn, kn, v, scratch, state, cu_seqlens, slot_ids, B, dm, o, st);
-    if (D <= 64) return launch_chunks<8>(qn, kn, v, scratch, state, cu_seqlens, slot_ids, B, dm, o, st);
-    if (D <= 128)
-      return launch_chunks<16>(qn, kn, v, scratch, state, cu_seqlens, slot_ids, B, dm, o, st);
-    return launch_chunks<32>(qn, kn, v, scratch, state, cu_seqlens, slot_ids, B, dm, o, st);
+#define GF_GO(DPER, LANES)                                                                         \
+  if (D <= DPER * LANES)                                                                           \
+    return launch_chunks<DPER, LANES>(qn, kn, v, scratch, state, cu_seqlens, slot_ids, B, dm, o, st);
+    GF_GO(4, 8)
+    GF_GO(8, 8)
+    GF_GO(16, 8)             // (sixteen lanes of 8 rows: 348 us for a prompt that takes 317 so)
+    GF_GO(16, 16)
+#undef GF_GO
   }
   // few (request, head, column) triples: a warp (sixteen lanes for key sizes up to 64) a column
   // instead of four lanes (see the kernel)

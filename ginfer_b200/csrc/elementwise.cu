@@ -313,14 +313,14 @@ int launch_add_rmsnorm(const void* x, const void* delta, const void* gamma, cons
 
 // Element-wise activations in place, fp32 arithmetic: kind 0 = relu(x)^2; kind 1 = a soft cap,
 // c * tanh(x / c); kind 2 = xIELU with the constants c and c2.  Four elements a pass where the count allows, the rest one by one.
-template <typename T>
-__global__ void activation_kernel(T* __restrict__ x, size_t total, int kind, float c, float c2) {
+template <typename T, int KIND>
+__global__ void activation_kernel(T* __restrict__ x, size_t total, float c, float c2) {
   pdl_trigger();
   pdl_wait();
   const size_t nq = (((uintptr_t)x % (4 * sizeof(T))) == 0) ? total / 4 : 0;
   auto f = [&](float v) {
-    if (kind == 0) { v = fmaxf(v, 0.f); return v * v; }
-    if (kind == 2) return xielu(v, c, c2);
+    if (KIND == 0) { v = fmaxf(v, 0.f); return v * v; }
+    if (KIND == 2) return xielu(v, c, c2);
     return c * tanhf(v / c);
   };
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < nq;
@@ -439,9 +439,16 @@ GF_EXPORT int gf_activation(void* x, long long total, int kind, float c, float c
   auto st = (cudaStream_t)stream;
   const size_t want = ((size_t)total / 4 + 255) / 256 + 1;
   const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
-  if (dtype == GF_F32)
-    return launch_kernel(activation_kernel<float>, dim3(blocks), dim3(256), 0, st, (float*)x,
-                         (size_t)total, kind, c, c2);
-  return launch_kernel(activation_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, st,
-                       (__nv_bfloat16*)x, (size_t)total, kind, c, c2);
+#define GF_GO(KIND)                                                                                \
+  if (kind == KIND && dtype == GF_F32)                                                             \
+    return launch_kernel(activation_kernel<float, KIND>, dim3(blocks), dim3(256), 0, st,           \
+                         (float*)x, (size_t)total, c, c2);                                         \
+  if (kind == KIND)                                                                                \
+    return launch_kernel(activation_kernel<__nv_bfloat16, KIND>, dim3(blocks), dim3(256), 0, st,   \
+                         (__nv_bfloat16*)x, (size_t)total, c, c2);
+  GF_GO(0)
+  GF_GO(1)
+  GF_GO(2)
+#undef GF_GO
+  return -3;
 }
