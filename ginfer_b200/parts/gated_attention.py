@@ -97,6 +97,8 @@ class NormedGatedAttention(Mixer):
                 or (self.position is not None and self.position.mult != 1.0):
             raise ValueError("norms without weights, values of another size than the keys and "
                              "stretched rotations go with norm_after_rotation")
+        if max(self.hd, self.vd) > 256:
+            raise ValueError(f"heads of {self.hd} | {self.vd} channels are over the attention kernels' 256")
         if self.vd != self.hd and not self.value_projection:
             raise ValueError("values that are the keys have the keys' size")
         # head sizes as the kernels see them (padded at load)

@@ -120,7 +120,7 @@ def test_a_run_must_name_the_state_its_block_keeps():
 
 
 def test_head_sizes_as_the_kernels_run_them():
-    assert [padded_head_size(*s) for s in ((16, 16), (32, 32), (16, 12), (32, 16), (64, 48), (48, 64),
+    assert [padded_head_size(*s) for s in ((16, 16), (32, 32), (16, 12), (32, 16), (60, 44), (40, 64),
                                            (64, 64), (65, 1), (128, 128), (96, 100), (129, 7),
                                            (256, 256), (257, 8))] == \
         [16, 32, 64, 64, 64, 64, 64, 128, 128, 128, 144, 256, 0]
@@ -145,7 +145,8 @@ def test_refused_combinations_of_attention_options():
     for bad in (dict(qk_norm_weights=False), dict(v_dim=4, value_projection=True),
                 dict(position=yarn), dict(norm_after_rotation=True),
                 dict(norm_after_rotation=True, qk_norm_weights=False, q_temp=(0.1, 4)),
-                dict(norm_after_rotation=True, qk_norm_weights=False, v_dim=4)):
+                dict(norm_after_rotation=True, qk_norm_weights=False, v_dim=4),
+                dict(head_dim=257)):
         with pytest.raises(ValueError):
             make_part("mixer", PartSpec("qknorm_attention", {**base, **bad}))
     with pytest.raises(ValueError, match="both"):

@@ -89,7 +89,7 @@ def row_errors(rows, want):
 # float32: differences of summation order.  bfloat16: the folders' peaked attention amplifies the
 # format's rounding, so single rows may be off (at most one in thirty) while the mean stays small;
 # a misplaced page, a lost state or a window off by one puts most rows near one.
-LIMIT = {"float32": (1e-4, 2e-5), "bfloat16": (0.3, 0.05)}
+LIMIT = {"float32": (5e-5, 1e-5), "bfloat16": (0.1, 0.02)}
 
 
 def check(rows, want, dtype, requests):
@@ -474,7 +474,7 @@ def test_shifted_norm_of_a_long_portion_and_a_wide_output_type_of_y():
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("nh, nkv, D, Vd, P, dims, yarn", [
-    (4, 2, 16, 12, None, 8, True), (3, 1, 24, 28, None, 24, True), (6, 2, 64, 48, 64, 32, True),
+    (4, 2, 16, 12, None, 8, True), (3, 1, 24, 28, None, 24, True), (6, 2, 56, 44, 64, 28, True),
     (5, 5, 14, 9, None, 6, False), (2, 1, 96, 80, 128, 48, True), (3, 3, 33, 8, None, 0, False),
     (16, 4, 128, 128, None, 64, True), (2, 2, 192, 160, None, 100, True), (4, 1, 40, 64, 64, 40, True)])
 def test_rotation_then_norm_of_heads_and_the_cache_write(dtype, nh, nkv, D, Vd, P, dims, yarn):
