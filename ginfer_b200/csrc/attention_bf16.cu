@@ -47,7 +47,7 @@ template <int MAXC>
 __device__ __forceinline__ void cluster_merge(float* cpart, float* cpart_m, float* cpart_l,
                                               float* cw, float* cinv, bf16* __restrict__ out,
                                               int nrows, int splits, int split, int row, int nh,
-                                              int h0, float sink, bool active = true,
+                                              int h0, const Sink sink, bool active = true,
                                               float* part_o = nullptr, float* part_ml = nullptr,
                                               int parts = 1) {
   // Loads from the peers are issued eight at a time without branches (the peer index is
@@ -73,7 +73,7 @@ __device__ __forceinline__ void cluster_merge(float* cpart, float* cpart_m, floa
       cw[r * 16 + p] = wgt;
       lsum += wgt * lp[p];
     }
-    cinv[r] = lsum > 0.f ? 1.f / (lsum + sink_share(sink, mm)) : 0.f;
+    cinv[r] = lsum > 0.f ? 1.f / (lsum + sink_share(sink.at(h0 + r), mm)) : 0.f;
     // part_o / part_ml: this cluster holds only a part of the request's keys; it leaves its
     // unnormalised result with the maximum and the sum for the kernel that merges the parts
     // (both pointers stand at this cluster's part of its first head; a head has `parts` parts)
@@ -340,7 +340,7 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16* __r
     const int head = h0 + r;
     if (splits == 1) {
       out[((size_t)row * nh + head) * HD + d] =
-          __float2bfloat16_rn(lsum > 0.f ? acc / (lsum + sink_share(shape.sink, mm)) : 0.f);
+          __float2bfloat16_rn(lsum > 0.f ? acc / (lsum + sink_share(shape.sink.at(head), mm)) : 0.f);
     } else if (fused_merge == 2) {
       cpart[i] = acc;                                   // this CTA's partial stays in shared memory
       if (d == 0) {
@@ -409,7 +409,7 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16* __r
       w[r * used + s2] = wgt;
       lsum += wgt * __ldcg(pml + (base + s2) * 2 + 1);
     }
-    linv[r] = lsum > 0.f ? 1.f / (lsum + sink_share(shape.sink, mm)) : 0.f;
+    linv[r] = lsum > 0.f ? 1.f / (lsum + sink_share(shape.sink.at(h0 + r), mm)) : 0.f;
   }
   __syncthreads();
   for (int i = threadIdx.x; i < nrows * HD; i += NTHREADS) {
@@ -472,7 +472,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap,
                        bf16* __restrict__ out, int nh, int nkv, int page_size, int window,
                        float scale_log2, int splits, int oob_row, int tbl_cap, int nst,
                        int* err, const RopeArgs rope, int parts, float* __restrict__ po,
-                       float* __restrict__ pml, float sink) {
+                       float* __restrict__ pml, const Sink sink) {
   // No static shared memory in this kernel: the dynamic part then starts at the aligned base,
   // which the swizzled tiles need (checked below: a misaligned base ends the CTA with code 5).
   extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -794,7 +794,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap,
       }
     } else if (splits == 1) {
       out[((size_t)row * nh + h0 + r) * HD + d] =
-          __float2bfloat16_rn(lsum > 0.f ? acc / (lsum + sink_share(sink, mm)) : 0.f);
+          __float2bfloat16_rn(lsum > 0.f ? acc / (lsum + sink_share(sink.at(h0 + r), mm)) : 0.f);
     } else {
       cpart[i] = acc;
       if (d == 0) {
@@ -823,7 +823,7 @@ __global__ void attn_decode_merge_kernel(const float* __restrict__ po,
                                          const float* __restrict__ pml,
                                          const int* __restrict__ cu_seqlens_q,
                                          bf16* __restrict__ out, int nh, int splits,
-                                         float sink) {
+                                         const Sink sink) {
   const int head = blockIdx.x, b = blockIdx.y, d = threadIdx.x;
   pdl_trigger();
   pdl_wait();
@@ -842,7 +842,7 @@ __global__ void attn_decode_merge_kernel(const float* __restrict__ po,
   }
   const int row = cu_seqlens_q ? cu_seqlens_q[b] : b;
   out[((size_t)row * nh + head) * HD + d] =
-      __float2bfloat16_rn(lsum > 0.f ? acc / (lsum + sink_share(sink, mm)) : 0.f);
+      __float2bfloat16_rn(lsum > 0.f ? acc / (lsum + sink_share(sink.at(head), mm)) : 0.f);
 }
 
 // ================================================================================== prefill
@@ -1031,7 +1031,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_row_stride, const bf16* __
       li += __shfl_xor_sync(0xffffffffu, li, 2);
       const int r = warp * WROWS + mt * 16 + g + 8 * i;
       if (r >= rows) continue;
-      const float inv = li > 0.f ? 1.f / (li + sink_share(shape.sink, m[mt][i])) : 0.f;
+      const float inv = li > 0.f ? 1.f / (li + sink_share(shape.sink.at(head), m[mt][i])) : 0.f;
       bf16* orow = out + ((size_t)(q_begin + r0 + r) * nh + head) * HD;
 #pragma unroll
       for (int n = 0; n < HD / 8; ++n) {
@@ -1064,7 +1064,7 @@ static int attn_decode_impl(const void* q, int q_row_stride, const void* kpages,
                             const int* cu_seqlens_q, const int* positions, void* out,
                             void* scratch, int B, int nh, int nkv, int page_size, int window,
                             float scale, int splits, const RopeArgs& rope, void* stream,
-                            const ScoreShape shape = ScoreShape{0.f, nullptr, kNoSink}) {
+                            const ScoreShape shape = ScoreShape{0.f, nullptr, Sink{kNoSink, nullptr}}) {
   if (B <= 0) return 0;
   if (nkv <= 0 || nh <= 0 || nh % nkv || splits < 1) return -3;
   auto st = (cudaStream_t)stream;
@@ -1127,14 +1127,14 @@ static int attn_decode_impl(const void* q, int q_row_stride, const void* kpages,
 // are a multiple of 8 and divide (or are a multiple of) the 64-key tile, 1 split or a cluster of
 // 2, 4, 8 or 16.  -6: not served (the caller takes gf_attn_decode / gf_attn_decode_rope).
 // `stages`: depth of the ring of tiles (2 .. 6, cut to what shared memory holds; 3 lets two CTAs
-// share an SM).  `sink`: the sink's score, -inf for none.  `err` receives 4 or 6 if a wait for a tile or for a free stage ran out.
+// share an SM).  `sink`: the sink's score, -inf for none; `sinks` (fp32 [nh] or null): one a head.  `err` receives 4 or 6 if a wait for a tile or for a free stage ran out.
 GF_EXPORT int gf_attn_decode_tma(const void* q, int q_row_stride, void* kpages, void* vpages,
                                  int num_pages, const int* block_table, int table_stride,
                                  const int* cu_seqlens_q, const int* positions, void* out, int B,
                                  int nh, int nkv, int page_size, int window, float scale,
                                  int splits, int stages, const float* rope_table, int rot,
                                  int fused, int write_kv, int* err, void* stream, int parts,
-                                 void* scratch, float sink) {
+                                 void* scratch, float sink, const float* sinks) {
 #if GF_HEAD_DIM % 64 == 0
   if (B <= 0) return 0;
   if (nh % nkv || splits < 1 || parts < 1 || (parts > 1 && !scratch)) return -3;
@@ -1183,10 +1183,10 @@ GF_EXPORT int gf_attn_decode_tma(const void* q, int q_row_stride, void* kpages, 
                                       (bf16*)kpages, (bf16*)vpages, block_table, table_stride,
                                       cu_seqlens_q, positions, (bf16*)out, nh, nkv, page_size,
                                       window, scale * LOG2E, splits, (int)slots, tbl_cap, nst, err,
-                                      rope, parts, po, pml, sink);
+                                      rope, parts, po, pml, Sink{sink, sinks});
   if (rc || parts == 1) return rc;
   return launch_kernel(attn_decode_merge_kernel, dim3(nh, B), dim3(HD), 0, st, (const float*)po,
-                       (const float*)pml, cu_seqlens_q, (bf16*)out, nh, parts, sink);
+                       (const float*)pml, cu_seqlens_q, (bf16*)out, nh, parts, Sink{sink, sinks});
 #else
   return -6;
 #endif
@@ -1219,18 +1219,19 @@ GF_EXPORT int gf_attn_decode_rope(const void* q, int q_row_stride, void* kpages,
 
 // gf_attn_decode with shaped scores: `softcap` > 0 caps them (cap * tanh(score / cap)), `slopes`
 // (fp32 [nh] or null) takes slope * (p - c) off the score of the key at c, `sink` (-inf: none) is
-// the score of a sink.
+// the score of a sink, `sinks` (fp32 [nh] or null) one a head.
 GF_EXPORT int gf_attn_decode_shaped(const void* q, int q_row_stride, const void* kpages,
                                     const void* vpages, const int* block_table, int table_stride,
                                     const int* cu_seqlens_q, const int* positions, void* out,
                                     void* scratch, int B, int nh, int nkv, int page_size,
                                     int window, float scale, int splits, float softcap,
-                                    const float* slopes, float sink, void* stream) {
+                                    const float* slopes, float sink, const float* sinks,
+                                    void* stream) {
   if (softcap < 0.f) return -3;
   return attn_decode_impl(q, q_row_stride, kpages, vpages, block_table, table_stride,
                           cu_seqlens_q, positions, out, scratch, B, nh, nkv, page_size, window,
                           scale, splits, RopeArgs{nullptr, 0, 0, 0}, stream,
-                          ScoreShape{softcap, slopes, sink});
+                          ScoreShape{softcap, slopes, Sink{sink, sinks}});
 }
 
 static int attn_prefill_impl(const void* q, int q_row_stride, const void* kpages,
@@ -1265,7 +1266,7 @@ GF_EXPORT int gf_attn_prefill(const void* q, int q_row_stride, const void* kpage
                               float scale, void* stream) {
   return attn_prefill_impl(q, q_row_stride, kpages, vpages, block_table, table_stride,
                            cu_seqlens_q, kv_lens, out, B, max_q_len, nh, nkv, page_size, window,
-                           scale, stream, ScoreShape{0.f, nullptr, kNoSink});
+                           scale, stream, ScoreShape{0.f, nullptr, Sink{kNoSink, nullptr}});
 }
 
 // The same with shaped scores (see gf_attn_decode_shaped).
@@ -1274,11 +1275,11 @@ GF_EXPORT int gf_attn_prefill_shaped(const void* q, int q_row_stride, const void
                                      const int* cu_seqlens_q, const int* kv_lens, void* out,
                                      int B, int max_q_len, int nh, int nkv, int page_size,
                                      int window, float scale, float softcap, const float* slopes,
-                                     float sink, void* stream) {
+                                     float sink, const float* sinks, void* stream) {
   if (softcap < 0.f) return -3;
   return attn_prefill_impl(q, q_row_stride, kpages, vpages, block_table, table_stride,
                            cu_seqlens_q, kv_lens, out, B, max_q_len, nh, nkv, page_size, window,
-                           scale, stream, ScoreShape{softcap, slopes, sink});
+                           scale, stream, ScoreShape{softcap, slopes, Sink{sink, sinks}});
 }
 
 // ----------------------------------------------------------------------------- no allocation

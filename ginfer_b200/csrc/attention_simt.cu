@@ -22,7 +22,7 @@ __global__ void paged_attention_simt_kernel(
     const T* __restrict__ vpages, const int* __restrict__ block_table, int table_stride,
     const int* __restrict__ seq_of_token, const int* __restrict__ positions, T* __restrict__ out,
     int num_pairs, int nh, int nkv, int hd, int vd, int page_size, int window, float scale,
-    float softcap, const float* __restrict__ slopes, float sink) {
+    float softcap, const float* __restrict__ slopes, const Sink sink) {
   extern __shared__ float qs_all[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int pair = blockIdx.x * kWarps + warp;
@@ -80,7 +80,7 @@ __global__ void paged_attention_simt_kernel(
     m = m_new;
   }
   T* orow = out + ((size_t)t * nh + n) * vd;
-  const float inv = 1.f / (l + expf(sink - m));    // no sink: exp(-inf) = 0
+  const float inv = 1.f / (l + expf(sink.at(n) - m));    // no sink: exp(-inf) = 0
 #pragma unroll
   for (int i = 0; i < kMaxHeadDim / 32; ++i) {
     const int d = lane + 32 * i;
@@ -97,14 +97,14 @@ GF_DEFINE_PDL_SWITCH
 // q: rows of q_row_stride elements whose first nh*hd hold the query heads.  kpages/vpages:
 // [num_pages, page_size, nkv, hd] and [.., nkv, vd].  out: [T, nh, vd] packed.  window: the mask as
 // first_visible_key() reads it.  softcap <= 0: no cap; slopes: nh fp32 slopes or null; sink: the
-// sink's score, -inf for none.  Returns -3
-// for head sizes it refuses.
+// sink's score, -inf for none; sinks: nh fp32 scores, one a head, or null.  Returns -3 for head sizes
+// it refuses.
 GF_EXPORT int gf_paged_attention_simt(const void* q, int q_row_stride, const void* kpages,
                                       const void* vpages, const int* block_table, int table_stride,
                                       const int* seq_of_token, const int* positions, void* out,
                                       int T, int nh, int nkv, int hd, int vd, int page_size,
                                       int window, float scale, float softcap, const float* slopes,
-                                      float sink, int dtype, void* stream) {
+                                      float sink, const float* sinks, int dtype, void* stream) {
   if (T <= 0) return 0;
   if (hd > kMaxHeadDim || hd <= 0 || vd > kMaxHeadDim || vd <= 0 || nh % nkv) return -3;
   const int pairs = T * nh;
@@ -115,11 +115,13 @@ GF_EXPORT int gf_paged_attention_simt(const void* q, int q_row_stride, const voi
     paged_attention_simt_kernel<float><<<blocks, kWarps * 32, smem, st>>>(
         (const float*)q, q_row_stride, (const float*)kpages, (const float*)vpages, block_table,
         table_stride, seq_of_token, positions, (float*)out, pairs, nh, nkv, hd, vd, page_size,
-        window, scale, softcap, slopes, sink);
+        window, scale, softcap, slopes,
+        Sink{sink, sinks});
   else
     paged_attention_simt_kernel<__nv_bfloat16><<<blocks, kWarps * 32, smem, st>>>(
         (const __nv_bfloat16*)q, q_row_stride, (const __nv_bfloat16*)kpages,
         (const __nv_bfloat16*)vpages, block_table, table_stride, seq_of_token, positions,
-        (__nv_bfloat16*)out, pairs, nh, nkv, hd, vd, page_size, window, scale, softcap, slopes, sink);
+        (__nv_bfloat16*)out, pairs, nh, nkv, hd, vd, page_size, window, scale, softcap, slopes,
+        Sink{sink, sinks});
   return launch_status();
 }

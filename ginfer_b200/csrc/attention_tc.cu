@@ -833,7 +833,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       const float f_me = m_used == -INFINITY ? 0.f : fast_exp2(m_used - m_all);
       const float f_o = m_o == -INFINITY ? 0.f : fast_exp2(m_o - m_all);
       const float l_all = l * f_me + l_o * f_o;
-      const float inv = l_all > 0.f ? 1.f / (l_all + sink_share(shape.sink, m_all)) : 0.f;
+      const float inv = l_all > 0.f ? 1.f / (l_all + sink_share(shape.sink.at(head), m_all)) : 0.f;
       // this stream writes channels s * HD / 2 .. of the row: from O_0 and (if stream 1 had a
       // tile at all) O_1, each with its stream's factor
       const float f0 = (s == 0 ? f_me : f_o) * inv, f1 = (s == 0 ? f_o : f_me) * inv;
@@ -983,22 +983,23 @@ GF_EXPORT int gf_attn_prefill_tc(const void* q, int q_row_stride, const void* kp
   return attn_prefill_tc_impl(q, q_row_stride, kpages, vpages, num_pages, block_table,
                               table_stride, cu_seqlens_q, kv_lens, out, T, B, max_q_len, nh, nkv,
                               page_size, window, scale, err, dbg, stream,
-                              ScoreShape{0.f, nullptr, kNoSink});
+                              ScoreShape{0.f, nullptr, Sink{kNoSink, nullptr}});
 }
 
 // The same with shaped scores: `softcap` > 0 caps them (cap * tanh(score / cap)); `slopes` (fp32
 // [nh] or null) takes slope * (p - c) off the score of the key at c for the query at p;
-// `sink` (-inf: none) is the score of a sink.
+// `sink` (-inf: none) is the score of a sink, `sinks` (fp32 [nh] or null) one a head.
 GF_EXPORT int gf_attn_prefill_tc_shaped(const void* q, int q_row_stride, const void* kpages,
                                         const void* vpages, int num_pages, const int* block_table,
                                         int table_stride, const int* cu_seqlens_q,
                                         const int* kv_lens, void* out, int T, int B, int max_q_len,
                                         int nh, int nkv, int page_size, int window, float scale,
-                                        float softcap, const float* slopes, float sink, int* err,
-                                        void* dbg, void* stream) {
+                                        float softcap, const float* slopes, float sink,
+                                        const float* sinks, int* err, void* dbg,
+                                        void* stream) {
   if (softcap < 0.f) return -3;
   return attn_prefill_tc_impl(q, q_row_stride, kpages, vpages, num_pages, block_table,
                               table_stride, cu_seqlens_q, kv_lens, out, T, B, max_q_len, nh, nkv,
                               page_size, window, scale, err, dbg, stream,
-                              ScoreShape{softcap, slopes, sink});
+                              ScoreShape{softcap, slopes, Sink{sink, sinks}});
 }

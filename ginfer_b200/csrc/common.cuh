@@ -112,12 +112,18 @@ __host__ __device__ __forceinline__ int first_visible_key(int p, int span) {
 // slopes (one a head), slope * (p - c) is then taken off the score of the key at c for the query at
 // p.  A sink adds exp(sink) to the softmax's denominator: a key with this score and no value.
 // 32-bit arithmetic in every kernel that takes it.
+constexpr float kNoSink = -__builtin_inff();
+// The sink's score: one for all heads (kNoSink: none), or one a head.
+struct Sink {
+  float score;
+  const float* heads;     // [heads], or null: `score` is every head's
+  __device__ __forceinline__ float at(int head) const { return heads ? heads[head] : score; }
+};
 struct ScoreShape {
   float cap;              // 0: no cap
   const float* slopes;    // [heads], or null: no distance bias
-  float sink;             // the sink's score; kNoSink: none
+  Sink sink;
 };
-constexpr float kNoSink = -__builtin_inff();
 // Whether single scores change (the sink only enters a row's sum, at its end).
 __host__ __device__ __forceinline__ bool shaped(const ScoreShape& sh) {
   return sh.cap > 0.f || sh.slopes != nullptr;

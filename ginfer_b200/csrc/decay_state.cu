@@ -22,9 +22,16 @@
 //                             and leave it four floats a load.  Lanes of a warp are laid out
 //                             [LP][32 / LP columns], so that a row of S is read and written in
 //                             whole 32-byte sectors (LP = 4).
+//                             With a NORMALISER the key rows are summed up by the same recurrence (a
+//                             column of the state whose value is always one), n_t = g_t n_(t-1) + c_t
+//                             k_t, and read out beside the others, n_t . q_t.
+//   memory_gates_kernel       the decays and step factors of a memory with exponential gates: a running
+//                             maximum m of the gates' logarithms (an associative scan over the
+//                             portion, carried in the slot) keeps every factor at or below one.
 //   gated_norm_kernel         a warp a (token, group of channels): RMS norm with a gate, the gate
 //                             before the norm (y = o silu(z), then y / rms(y) w) or behind it
-//                             (o / rms(o) w silu(z)); the weight per channel or shared by the groups.
+//                             (o / rms(o) w silu(z)); the weight per channel or shared by the groups
+//                             or none.  A group may first be divided by its normaliser's read-out.
 //   gated_norm_warp_vec_kernel  the same with four channels an access;
 //   gated_norm_block_kernel   the same with a block a (token, group), for groups over 512 channels;
 //   gated_norm_vec_kernel     with four channels an access and up to 1,024 threads where rows allow.
@@ -178,12 +185,71 @@ __global__ void silu_f32_vec_kernel(const __nv_bfloat16* __restrict__ proj, int 
   dst[1] = make_float4(z[4], z[5], z[6], z[7]);
 }
 
+// ------------------------------------------------------------------------------- exponential gates
+// A token's gates, per head: i = cap tanh((z_i + b_i) / cap), f = log sigmoid(cap tanh((z_f + b_f) /
+// cap)).  The running maximum m_t = max(f_t + m_(t-1), i_t) starts at the slot's (zero for a new
+// sequence); out: the decay exp(f_t + m_(t-1) - m_t), the factor exp(i_t - m_t) and m_t, [T, H] each.
+// A block a (head, request): a thread a token at a time, blockDim tokens together by a scan over the
+// maps m -> max(m + a, b), which compose to the same form.  Only m's own value depends on the order of
+// the sums; the factors are formed from the m that are written, so they fit together exactly.
+constexpr int kGateThreads = 256;
+__global__ void __launch_bounds__(kGateThreads)
+memory_gates_kernel(const float* __restrict__ proj, int ld, int i_col, int f_col,
+                    const float* __restrict__ i_bias, const float* __restrict__ f_bias, float cap,
+                    float* __restrict__ state, int state_stride, int m_off,
+                    const int* __restrict__ cu_seqlens, const int* __restrict__ slot_ids, int H,
+                    float* __restrict__ decay, float* __restrict__ factor,
+                    float* __restrict__ maxima, int early) {
+  __shared__ float wa[kGateThreads / 32], wb[kGateThreads / 32], last[kGateThreads];
+  const int h = blockIdx.x, b = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  if (early) pdl_trigger();
+  const float bi = i_bias[h], bfg = f_bias[h];
+  pdl_wait();
+  const int start = cu_seqlens[b], n = cu_seqlens[b + 1] - start;
+  float* slot = state + (size_t)slot_ids[b] * state_stride + m_off + h;
+  float m0 = *slot;
+  for (int t0 = 0; t0 < n; t0 += blockDim.x) {
+    const int t = t0 + threadIdx.x;
+    float gi = -INFINITY, gf = 0.f;                // past the end: the identity map
+    if (t < n) {
+      const float* row = proj + (size_t)(start + t) * ld;
+      gi = cap * tanhf((row[i_col + h] + bi) / cap);
+      gf = ds_log_sigmoid(cap * tanhf((row[f_col + h] + bfg) / cap));
+    }
+    float A = gf, B = gi;
+#pragma unroll
+    for (int off = 1; off < 32; off <<= 1) {
+      const float pa = __shfl_up_sync(0xffffffffu, A, off), pb = __shfl_up_sync(0xffffffffu, B, off);
+      if (lane >= off) B = fmaxf(pb + A, B), A += pa;
+    }
+    if (lane == 31) wa[warp] = A, wb[warp] = B;
+    __syncthreads();
+    float m_in = m0;                               // m in front of this warp's tokens
+    for (int w = 0; w < warp; ++w) m_in = fmaxf(m_in + wa[w], wb[w]);
+    const float m = fmaxf(m_in + A, B);
+    last[threadIdx.x] = m;
+    __syncthreads();
+    const float before = threadIdx.x == 0 ? m0 : last[threadIdx.x - 1];
+    if (t < n) {
+      const size_t at = (size_t)(start + t) * H + h;
+      decay[at] = expf(gf + before - m);
+      factor[at] = expf(gi - m);
+      maxima[at] = m;
+    }
+    m0 = last[min((int)blockDim.x, n - t0) - 1];
+    __syncthreads();
+  }
+  if (threadIdx.x == 0) *slot = m0;
+}
+
 // ------------------------------------------------------------------------------- the recurrence
 struct DecayDims {
   int H, G, D, Vd;
   int gD;                // D: a decay a key channel; 1: a decay a head
   int ld_q, ld_k, ld_v, ld_g, ld_c;   // floats between the rows of two tokens
   int state_stride;
+  int norm_off;          // where the normalisers [H, D] start in a slot; < 0: none
+  int ld_n;              // floats between the rows of two tokens' normaliser read-outs
 };
 
 __device__ __forceinline__ void ds_copy4(float* dst, const float* src) {
@@ -212,7 +278,7 @@ decay_recurrence_kernel(const float* __restrict__ q, const float* __restrict__ k
                         const float* __restrict__ c, const float* __restrict__ skip,
                         float* __restrict__ state, const int* __restrict__ cu_seqlens,
                         const int* __restrict__ slot_ids, DecayDims dm, float* __restrict__ o,
-                        int ld_o) {
+                        int ld_o, float* __restrict__ o_norm) {
   constexpr int CW = 32 / LP;                      // columns a warp
   constexpr int VT = kDecayWarps * CW;             // columns a block
   constexpr int DP = DPER * LP;                    // key channels, padded
@@ -225,22 +291,27 @@ decay_recurrence_kernel(const float* __restrict__ q, const float* __restrict__ k
   const int col0 = blockIdx.x * VT;
   const int col = col0 + warp * CW + vc;
   const int D = dm.D, Vd = dm.Vd, gk = h / (dm.H / dm.G);
-  const bool live = col < Vd, perch = dm.gD != 1;
+  // the column behind the values, where there is a normaliser: its value is one
+  const bool unit = dm.norm_off >= 0 && col == Vd;
+  const bool live = col < Vd || unit, perch = dm.gD != 1;
   // what cp.async never writes stays zero for ever: the padding rows of q, k and the decays, and
   // the columns past the last one
   for (int i = threadIdx.x; i < 2 * kDecayChunk * ROW; i += blockDim.x) {
     const int e = i % ROW;
     if (e >= 3 * DP || (e % DP) >= D) stage[i] = 0.f;
+    if (dm.norm_off >= 0 && e == 3 * DP + Vd - col0 && e < 3 * DP + VT) stage[i] = 1.f;
   }
   pdl_trigger();
   pdl_wait();
   const int start = cu_seqlens[b], n = cu_seqlens[b + 1] - start;
-  float* S = state + (size_t)slot_ids[b] * dm.state_stride + (size_t)h * D * Vd;
+  float* S = state + (size_t)slot_ids[b] * dm.state_stride +
+             (unit ? (size_t)dm.norm_off + (size_t)h * D : (size_t)h * D * Vd + col);
+  const int S_row = unit ? 1 : Vd;                 // floats between two rows of the column
   float s[DPER];
 #pragma unroll
   for (int i = 0; i < DPER; ++i) {
     const int d = lp * DPER + i;
-    s[i] = (live && d < D) ? S[(size_t)d * Vd + col] : 0.f;
+    s[i] = (live && d < D) ? S[(size_t)d * S_row] : 0.f;
   }
   const float sk = skip != nullptr ? skip[h] : 0.f;
   __syncthreads();
@@ -315,7 +386,9 @@ decay_recurrence_kernel(const float* __restrict__ q, const float* __restrict__ k
     if (ch + 1 < chunks) fetch(ch + 1, (ch + 1) & 1);
     const float* base = stage + (size_t)(ch & 1) * kDecayChunk * ROW;
     const int cnt = min(kDecayChunk, n - ch * kDecayChunk);
-    float* orow = o + (size_t)(start + ch * kDecayChunk) * ld_o + (size_t)h * Vd + col;
+    const int ldo = unit ? dm.ld_n : ld_o;
+    float* orow = unit ? o_norm + (size_t)(start + ch * kDecayChunk) * ldo + h
+                       : o + (size_t)(start + ch * kDecayChunk) * ldo + (size_t)h * Vd + col;
     int t = 0;
     for (; t + kDecayUnroll <= cnt; t += kDecayUnroll) {
       float acc[kDecayUnroll], vv[kDecayUnroll];
@@ -328,31 +401,43 @@ decay_recurrence_kernel(const float* __restrict__ q, const float* __restrict__ k
       if (lp == 0 && live)
 #pragma unroll
         for (int u = 0; u < kDecayUnroll; ++u)
-          orow[(size_t)(t + u) * ld_o] = fmaf(sk, vv[u], acc[u]);
+          orow[(size_t)(t + u) * ldo] = fmaf(sk, vv[u], acc[u]);
     }
     for (; t < cnt; ++t) {
       float vv;
       float acc = advance(base + t * ROW, vv);
 #pragma unroll
       for (int off = CW; off < 32; off <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, off);
-      if (lp == 0 && live) orow[(size_t)t * ld_o] = fmaf(sk, vv, acc);
+      if (lp == 0 && live) orow[(size_t)t * ldo] = fmaf(sk, vv, acc);
     }
   }
 #pragma unroll
   for (int i = 0; i < DPER; ++i) {
     const int d = lp * DPER + i;
-    if (live && d < D) S[(size_t)d * Vd + col] = s[i];
+    if (live && d < D) S[(size_t)d * S_row] = s[i];
   }
 }
 
 // ------------------------------------------------------------------------------- gated norm
+// What a group is multiplied by before anything else: scale / (max(|scale * n|, exp(-m)) + floor) with
+// n the read-out of its normaliser and m the running maximum its factors were kept below one with.
+struct Normaliser {
+  const float* n;           // [units], or null: nothing
+  const float* m;           // [units]
+  float scale, floor;
+  __device__ __forceinline__ float factor(int unit) const {
+    return n == nullptr ? 1.f
+                        : scale / (fmaxf(fabsf(scale * n[unit]), expf(-m[unit])) + floor);
+  }
+};
+
 // o [rows, C] fp32; gate [rows, ...] (G = float or bf16) with row stride gate_ld; groups of gs
 // channels; w [C] or, shared, [gs].
 template <typename G, typename T>
 __global__ void gated_norm_kernel(const float* __restrict__ o, const G* __restrict__ gate,
                                   int gate_ld, const float* __restrict__ w, int w_shared,
                                   int gate_mode, float eps, T* __restrict__ out, int units,
-                                  int groups, int gs) {
+                                  int groups, int gs, const Normaliser nrm) {
   const int unit = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   const int sig = gate_mode >> 1, gate_first = gate_mode & 1;
   pdl_trigger();
@@ -362,9 +447,10 @@ __global__ void gated_norm_kernel(const float* __restrict__ o, const G* __restri
   const float* orow = o + (size_t)r * groups * gs + (size_t)gi * gs;
   const G* grow = gate + (size_t)r * gate_ld + (size_t)gi * gs;
   T* dst = out + (size_t)r * groups * gs + (size_t)gi * gs;
+  const float nf = nrm.factor(unit);
   float ss = 0.f;
   for (int j = lane; j < gs; j += 32) {
-    float y = orow[j];
+    float y = orow[j] * nf;
     if (gate_first) {
       const float z = to_f32(grow[j]);
       y *= ds_gate(z, sig);
@@ -376,8 +462,8 @@ __global__ void gated_norm_kernel(const float* __restrict__ o, const G* __restri
   for (int j = lane; j < gs; j += 32) {
     const float z = to_f32(grow[j]);
     const float gz = ds_gate(z, sig);
-    const float wj = w[w_shared ? j : gi * gs + j];
-    const float y = gate_first ? orow[j] * gz * inv * wj : orow[j] * inv * wj * gz;
+    const float wj = w ? w[w_shared ? j : gi * gs + j] : 1.f;
+    const float y = gate_first ? orow[j] * nf * gz * inv * wj : orow[j] * nf * inv * wj * gz;
     dst[j] = from_f32<T>(y);
   }
 }
@@ -389,7 +475,7 @@ template <typename G, typename T, int NQ>
 __global__ void gated_norm_warp_vec_kernel(const float* __restrict__ o, const G* __restrict__ gate,
                                            int gate_ld, const float* __restrict__ w, int w_shared,
                                            int gate_mode, float eps, T* __restrict__ out, int units,
-                                           int groups, int gs) {
+                                           int groups, int gs, const Normaliser nrm) {
   const int unit = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   const int sig = gate_mode >> 1, gate_first = gate_mode & 1;
   pdl_trigger();
@@ -400,6 +486,7 @@ __global__ void gated_norm_warp_vec_kernel(const float* __restrict__ o, const G*
   const G* grow = gate + (size_t)r * gate_ld + (size_t)gi * gs;
   const float* wrow = w + (w_shared ? 0 : (size_t)gi * gs);
   T* dst = out + (size_t)r * groups * gs + (size_t)gi * gs;
+  const float nf = nrm.factor(unit);
   float y[NQ][4], z[NQ][4];
   float ss = 0.f;
 #pragma unroll
@@ -410,6 +497,7 @@ __global__ void gated_norm_warp_vec_kernel(const float* __restrict__ o, const G*
       Quad<G>::load(grow + 4 * q, z[u]);
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
+        y[u][i] *= nf;
         z[u][i] = ds_gate(z[u][i], sig);
         if (gate_first) y[u][i] *= z[u][i];
         ss = fmaf(y[u][i], y[u][i], ss);
@@ -422,8 +510,8 @@ __global__ void gated_norm_warp_vec_kernel(const float* __restrict__ o, const G*
   for (int u = 0; u < NQ; ++u) {
     const int q = lane + 32 * u;
     if (q < nq) {
-      float wq[4];
-      Quad<float>::load(wrow + 4 * q, wq);
+      float wq[4] = {1.f, 1.f, 1.f, 1.f};
+      if (w) Quad<float>::load(wrow + 4 * q, wq);
 #pragma unroll
       for (int i = 0; i < 4; ++i) y[u][i] *= gate_first ? inv * wq[i] : inv * wq[i] * z[u][i];
       Quad<T>::store(dst + 4 * q, y[u]);
@@ -436,7 +524,7 @@ template <typename G, typename T>
 __global__ void __launch_bounds__(256)
 gated_norm_block_kernel(const float* __restrict__ o, const G* __restrict__ gate, int gate_ld,
                         const float* __restrict__ w, int w_shared, int gate_mode, float eps,
-                        T* __restrict__ out, int groups, int gs) {
+                        T* __restrict__ out, int groups, int gs, const Normaliser nrm) {
   __shared__ float scratch[33];
   const int unit = blockIdx.x;
   const int sig = gate_mode >> 1, gate_first = gate_mode & 1;
@@ -446,9 +534,10 @@ gated_norm_block_kernel(const float* __restrict__ o, const G* __restrict__ gate,
   const float* orow = o + (size_t)r * groups * gs + (size_t)gi * gs;
   const G* grow = gate + (size_t)r * gate_ld + (size_t)gi * gs;
   T* dst = out + (size_t)r * groups * gs + (size_t)gi * gs;
+  const float nf = nrm.factor(unit);
   float ss = 0.f;
   for (int j = threadIdx.x; j < gs; j += blockDim.x) {
-    float y = orow[j];
+    float y = orow[j] * nf;
     if (gate_first) {
       const float z = to_f32(grow[j]);
       y *= ds_gate(z, sig);
@@ -460,8 +549,8 @@ gated_norm_block_kernel(const float* __restrict__ o, const G* __restrict__ gate,
   for (int j = threadIdx.x; j < gs; j += blockDim.x) {
     const float z = to_f32(grow[j]);
     const float gz = ds_gate(z, sig);
-    const float wj = w[w_shared ? j : gi * gs + j];
-    const float y = gate_first ? orow[j] * gz * inv * wj : orow[j] * inv * wj * gz;
+    const float wj = w ? w[w_shared ? j : gi * gs + j] : 1.f;
+    const float y = gate_first ? orow[j] * nf * gz * inv * wj : orow[j] * nf * inv * wj * gz;
     dst[j] = from_f32<T>(y);
   }
 }
@@ -473,7 +562,7 @@ template <typename G, typename T>
 __global__ void __launch_bounds__(1024)
 gated_norm_vec_kernel(const float* __restrict__ o, const G* __restrict__ gate, int gate_ld,
                       const float* __restrict__ w, int w_shared, int gate_mode, float eps,
-                      T* __restrict__ out, int groups, int gs) {
+                      T* __restrict__ out, int groups, int gs, const Normaliser nrm) {
   __shared__ float scratch[33];
   const int unit = blockIdx.x, nq = gs >> 2;
   const int sig = gate_mode >> 1, gate_first = gate_mode & 1;
@@ -484,10 +573,13 @@ gated_norm_vec_kernel(const float* __restrict__ o, const G* __restrict__ gate, i
   const G* grow = gate + (size_t)r * gate_ld + (size_t)gi * gs;
   const float* wrow = w + (w_shared ? 0 : (size_t)gi * gs);
   T* dst = out + (size_t)r * groups * gs + (size_t)gi * gs;
+  const float nf = nrm.factor(unit);
   float ss = 0.f;
   for (int q = threadIdx.x; q < nq; q += blockDim.x) {
     float y[4];
     Quad<float>::load(orow + 4 * q, y);
+#pragma unroll
+    for (int u = 0; u < 4; ++u) y[u] *= nf;
     if (gate_first) {
       float z[4];
       Quad<G>::load(grow + 4 * q, z);
@@ -500,12 +592,13 @@ gated_norm_vec_kernel(const float* __restrict__ o, const G* __restrict__ gate, i
   ss = block_sum(ss, scratch);
   const float inv = 1.f / sqrtf(ss / (float)gs + eps);
   for (int q = threadIdx.x; q < nq; q += blockDim.x) {
-    float y[4], z[4], wq[4];
+    float y[4], z[4], wq[4] = {1.f, 1.f, 1.f, 1.f};
     Quad<float>::load(orow + 4 * q, y);
     Quad<G>::load(grow + 4 * q, z);
-    Quad<float>::load(wrow + 4 * q, wq);
+    if (w) Quad<float>::load(wrow + 4 * q, wq);
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
+      y[u] *= nf;
       const float gz = ds_gate(z[u], sig);
       y[u] = gate_first ? y[u] * gz * inv * wq[u] : y[u] * inv * wq[u] * gz;
     }
@@ -586,23 +679,26 @@ GF_EXPORT int gf_silu_f32(const void* proj, int ld, int T, int width, float* out
 // q, k: rows of G heads of D; v: rows of H heads of Vd; g: rows of H x gD decays (gD = D or 1);
 // c: rows of H factors on k, or null; skip: H weights of v in the output, or null; state: the
 // slots, S [H, D, Vd] first in each.  wide: sixteen lanes a column instead of four (few requests
-// with long portions).  Returns -3 for key sizes over 256.
+// with long portions).  o_norm [.., H] (row stride ld_n): the normalisers' read-outs, whose sums [H, D]
+// start at norm_off in a slot; null: none.  Returns -3 for key sizes over 256.
 GF_EXPORT int gf_decay_recurrence(const float* q, int ld_q, const float* k, int ld_k,
                                   const float* v, int ld_v, const float* g, int ld_g, int gD,
                                   const float* c, int ld_c, const float* skip, float* state,
                                   int state_stride, const int* cu_seqlens, const int* slot_ids,
                                   int B, int H, int G, int D, int Vd, float* o, int ld_o, int wide,
-                                  void* stream) {
+                                  int norm_off, float* o_norm, int ld_n, void* stream) {
   if (B <= 0) return 0;
   if (G <= 0 || H % G || (gD != 1 && gD != D) || D <= 0 || D > 256) return -3;
   DecayDims dm;
   dm.H = H, dm.G = G, dm.D = D, dm.Vd = Vd, dm.gD = gD;
   dm.ld_q = ld_q, dm.ld_k = ld_k, dm.ld_v = ld_v, dm.ld_g = ld_g, dm.ld_c = ld_c;
   dm.state_stride = state_stride;
+  dm.norm_off = o_norm != nullptr ? norm_off : -1, dm.ld_n = ld_n;
+  if (o_norm != nullptr && (norm_off < 0 || skip != nullptr)) return -2;
   auto st = (cudaStream_t)stream;
   const int lp = wide ? 16 : 4;
   const int vt = kDecayWarps * (32 / lp);
-  const dim3 grid((Vd + vt - 1) / vt, H, B), block(kDecayWarps * 32);
+  const dim3 grid((Vd + (o_norm != nullptr) + vt - 1) / vt, H, B), block(kDecayWarps * 32);
   auto aligned = [](const float* p, int ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; };
   const bool vec = D % 4 == 0 && Vd % 4 == 0 && aligned(q, ld_q) && aligned(k, ld_k) &&
                    aligned(v, ld_v) && (gD == 1 || aligned(g, ld_g));
@@ -617,7 +713,7 @@ GF_EXPORT int gf_decay_recurrence(const float* q, int ld_q, const float* k, int 
     });                                                                                            \
     if (rc) return rc;                                                                             \
     return launch_kernel(decay_recurrence_kernel<DPER, LP, VEC>, grid, block, smem, st, q, k, v,   \
-                         g, c, skip, state, cu_seqlens, slot_ids, dm, o, ld_o);                    \
+                         g, c, skip, state, cu_seqlens, slot_ids, dm, o, ld_o, o_norm);            \
   }
 #define GF_GO(DPER, LP)                                                                            \
   if (lp == LP && D <= LP * DPER) {                                                                \
@@ -641,9 +737,14 @@ GF_EXPORT int gf_decay_recurrence(const float* q, int ld_q, const float* k, int 
 
 // o: [T, groups * gs] fp32 -> out in the activation dtype.  gate_dtype: the gate's own.
 // gate_first: bit 0 = the gate before the norm; bit 1 = the gate is sigmoid(z), not z sigmoid(z).
+// w null: no weight.  norm_read, norm_max [T, groups] (norm_read null: none): see Normaliser.
 GF_EXPORT int gf_gated_norm(const float* o, const void* gate, int gate_ld, int gate_dtype,
                             const float* w, int w_shared, int gate_first, float eps, void* out,
-                            int T, int groups, int gs, int dtype, void* stream) {
+                            int T, int groups, int gs, const float* norm_read,
+                            const float* norm_max, float norm_scale, float norm_floor, int dtype,
+                            void* stream) {
+  if (norm_read && !norm_max) return -2;
+  const Normaliser nrm{norm_read, norm_max, norm_scale, norm_floor};
   const int units = T * groups;
   if (units <= 0) return 0;
   auto st = (cudaStream_t)stream;
@@ -659,25 +760,40 @@ GF_EXPORT int gf_gated_norm(const float* o, const void* gate, int gate_ld, int g
     if (vec)                                                                                       \
       return launch_kernel(gated_norm_vec_kernel<GT, OT>, dim3(units), dim3(vthreads), 0, st, o,   \
                            (const GT*)gate, gate_ld, w, w_shared, gate_first, eps, (OT*)out,       \
-                           groups, gs);                                                            \
+                           groups, gs, nrm);                                                       \
     if (!wide && quad_rows && gs <= 128)                                                           \
       return launch_kernel(gated_norm_warp_vec_kernel<GT, OT, 1>, grid, block, 0, st, o,           \
                            (const GT*)gate, gate_ld, w, w_shared, gate_first, eps, (OT*)out,       \
-                           units, groups, gs);                                                     \
+                           units, groups, gs, nrm);                                                \
     if (!wide && quad_rows)                                                                        \
       return launch_kernel(gated_norm_warp_vec_kernel<GT, OT, 4>, grid, block, 0, st, o,           \
                            (const GT*)gate, gate_ld, w, w_shared, gate_first, eps, (OT*)out,       \
-                           units, groups, gs);                                                     \
+                           units, groups, gs, nrm);                                                \
     if (wide)                                                                                      \
       return launch_kernel(gated_norm_block_kernel<GT, OT>, dim3(units), dim3(256), 0, st, o,      \
                            (const GT*)gate, gate_ld, w, w_shared, gate_first, eps, (OT*)out,       \
-                           groups, gs);                                                            \
+                           groups, gs, nrm);                                                       \
     return launch_kernel(gated_norm_kernel<GT, OT>, grid, block, 0, st, o, (const GT*)gate,        \
-                         gate_ld, w, w_shared, gate_first, eps, (OT*)out, units, groups, gs);      \
+                         gate_ld, w, w_shared, gate_first, eps, (OT*)out, units, groups, gs, nrm); \
   }
   if (gate_dtype == GF_F32 && dtype == GF_F32) GF_GO(float, float)
   if (gate_dtype == GF_F32) GF_GO(float, bf)
   if (dtype == GF_F32) GF_GO(bf, float)
   GF_GO(bf, bf)
 #undef GF_GO
+}
+
+// proj: rows of ld floats with the H input gates from i_col and the H forget gates from f_col on; the
+// running maxima [H] start at m_off in a slot.  early: see gf_rotary_heads.
+GF_EXPORT int gf_memory_gates(const float* proj, int ld, int i_col, int f_col, const float* i_bias,
+                              const float* f_bias, float cap, float* state, int state_stride,
+                              int m_off, const int* cu_seqlens, const int* slot_ids, int B, int H,
+                              int max_q_len, float* decay, float* factor, float* maxima, int early,
+                              void* stream) {
+  if (B <= 0) return 0;
+  if (!(cap > 0.f)) return -3;
+  const int threads = max_q_len >= kGateThreads ? kGateThreads : (max_q_len + 31) / 32 * 32;
+  return launch_kernel(memory_gates_kernel, dim3(H, B), dim3(threads), 0, (cudaStream_t)stream, proj,
+                       ld, i_col, f_col, i_bias, f_bias, cap, state, state_stride, m_off, cu_seqlens,
+                       slot_ids, H, decay, factor, maxima, early);
 }

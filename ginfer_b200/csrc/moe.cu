@@ -5,6 +5,10 @@
 //                       (or the sigmoid of each logit), the `top` largest chosen (lowest index
 //                       among equals), their scores kept as weights (optionally renormalised over
 //                       the chosen ones).
+//   moe_route_grouped_kernel  the same over groups of neighbouring experts, chosen by scores that a
+//                       correction shifts: only experts of the groups with the largest best score can be
+//                       chosen; the last outputs may be experts without matrices (identity), whose
+//                       weights are added up per token; the row may hold a gate's logit as well.
 //   moe_plan_kernel     a block an expert: (token, choice) pairs counted per expert, the experts' ranges in
 //                       the sorted order, each pair's place, and the list of row tiles (expert,
 //                       first row) that the grouped products walk over.
@@ -78,8 +82,109 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int T, int E,
   }
 }
 
+// logits: rows of ld floats, E router outputs first: E - identity experts with matrices, then the
+// identity ones.  Scores s = softmax over all E; choice scores c = s + correction (null: s).  groups > 1:
+// equal groups of E / groups neighbours, a group's score the largest c in it, the `keep` best groups
+// stay (lowest index among equals).  Of their experts the `top` with the largest c are chosen (lowest
+// index among equals).  idx: the expert, or -1 for an identity one; wgt: its s (0 for an identity one);
+// identity_w[t]: the sum of the identity ones' s (null: not wanted).  gate[t] = sigmoid(row[gate_col])
+// (null: no gate).
+__global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int ld, int T, int E,
+                                         int identity, int top, int groups, int keep,
+                                         const float* __restrict__ correction, int gate_col,
+                                         int* __restrict__ idx, float* __restrict__ wgt,
+                                         float* __restrict__ identity_w,
+                                         float* __restrict__ gate) {
+  constexpr int kW = 4;                                       // warps a block
+  __shared__ float gscore[kW][kMaxExperts];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * kW + warp;
+  pdl_trigger();
+  pdl_wait();
+  if (t >= T) return;                                         // (warps are independent)
+  const float* row = logits + (size_t)t * ld;
+  float s[kRouteSlots], c[kRouteSlots];
+  float mx = -INFINITY;
+#pragma unroll
+  for (int i = 0; i < kRouteSlots; ++i) {
+    const int e = lane + 32 * i;
+    s[i] = e < E ? row[e] : -INFINITY;
+    mx = fmaxf(mx, s[i]);
+  }
+  mx = warp_max(mx);
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < kRouteSlots; ++i) {
+    s[i] = expf(s[i] - mx);                                   // 0 past the last expert
+    sum += s[i];
+  }
+  sum = warp_sum(sum);
+#pragma unroll
+  for (int i = 0; i < kRouteSlots; ++i) {
+    const int e = lane + 32 * i;
+    s[i] = s[i] / sum;
+    c[i] = e < E ? s[i] + (correction ? correction[e] : 0.f) : -INFINITY;
+  }
+  if (groups > 1 && keep < groups) {
+    const int gs = E / groups;
+    float* gsc = gscore[warp];
+    for (int g = 0; g < groups; ++g) {
+      float best = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < kRouteSlots; ++i) {
+        const int e = lane + 32 * i;
+        if (e >= g * gs && e < (g + 1) * gs) best = fmaxf(best, c[i]);
+      }
+      best = warp_max(best);
+      if (lane == 0) gsc[g] = best;
+    }
+    __syncwarp();
+    // a group stays if fewer than `keep` groups come before it (larger, or equal with a lower index)
+#pragma unroll
+    for (int i = 0; i < kRouteSlots; ++i) {
+      const int e = lane + 32 * i;
+      if (e >= E) continue;
+      const int g = e / gs;
+      int ahead = 0;
+      for (int o = 0; o < groups; ++o) ahead += gsc[o] > gsc[g] || (gsc[o] == gsc[g] && o < g);
+      if (ahead >= keep) c[i] = -INFINITY;
+    }
+  }
+  const int E0 = E - identity;
+  float id_sum = 0.f;
+  for (int k = 0; k < top; ++k) {
+    float best = -INFINITY;
+    int be = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < kRouteSlots; ++i)
+      if (c[i] > best) best = c[i], be = lane + 32 * i;       // ascending e: lowest index wins
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+      if (ob > best || (ob == best && oe < be)) best = ob, be = oe;
+    }
+    float w = 0.f;
+#pragma unroll
+    for (int i = 0; i < kRouteSlots; ++i)
+      if (lane + 32 * i == be) w = s[i], c[i] = -INFINITY;
+    w = __shfl_sync(0xffffffffu, w, be & 31);
+    const bool none = be >= E0;                               // an identity expert (or none is left)
+    if (none) id_sum += w;
+    if (lane == 0) {
+      idx[(size_t)t * top + k] = none ? -1 : be;
+      wgt[(size_t)t * top + k] = none ? 0.f : w;
+    }
+  }
+  if (lane == 0) {
+    if (identity_w) identity_w[t] = id_sum;
+    if (gate) gate[t] = 1.f / (1.f + expf(-row[gate_col]));
+  }
+}
+
 // Pairs p = t * top + k.  offsets[E + 1]; pos_of_pair[P]; pair_of_pos[P]; tiles: tile_expert[],
-// tile_row0[] (first sorted row of the tile), num_tiles[0].
+// tile_row0[] (first sorted row of the tile), num_tiles[0].  A pair whose expert is -1 has no place
+// (pos_of_pair -1): the sorted order then holds offsets[E] < P pairs.
 // A block an expert (one SM could not keep up: 8,192 pairs took 29 us in one block).  Every block
 // counts all experts' pairs for itself, so that it knows where its expert's rows and tiles begin
 // without waiting for another block; then its warps take equal runs of the pairs, count their
@@ -144,6 +249,7 @@ moe_plan_kernel(const int* __restrict__ idx, int P, int E, int tile_rows,
       pair_of_pos[pos] = p;
     }
     at += __popc(m);
+    if (e == 0 && p < p_hi && idx[p] < 0) pos_of_pair[p] = -1;
   }
 }
 
@@ -496,11 +602,13 @@ moe_gemv_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_bfloat1
 // xs[s, :] = x[pair_of_pos[s] / top, :]: the tokens' rows in sorted order, 16 bytes an access, for
 // the grouped product that reads its rows by TMA (K % 8 == 0, 16-byte aligned rows).
 __global__ void moe_gather_rows_kernel(const __nv_bfloat16* __restrict__ x, int ldx,
-                                       const int* __restrict__ pair_of_pos, int top, int P, int K,
+                                       const int* __restrict__ pair_of_pos,
+                                       const int* __restrict__ placed, int top, int P, int K,
                                        __nv_bfloat16* __restrict__ xs) {
   pdl_trigger();
   pdl_wait();
   const int k8 = K >> 3;
+  P = min(P, *placed);                              // pairs that have a place
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < (size_t)P * k8;
        i += (size_t)gridDim.x * blockDim.x) {
     const size_t s = i / k8;
@@ -519,9 +627,10 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
   pdl_wait();
   for (int n = threadIdx.x; n < N; n += blockDim.x) {
     float acc = 0.f;
-    for (int k = 0; k < top; ++k)
-      acc = fmaf(wgt ? wgt[(size_t)t * top + k] : 1.f,
-                 y[(size_t)pos_of_pair[(size_t)t * top + k] * N + n], acc);
+    for (int k = 0; k < top; ++k) {
+      const int p = pos_of_pair[(size_t)t * top + k];
+      if (p >= 0) acc = fmaf(wgt ? wgt[(size_t)t * top + k] : 1.f, y[(size_t)p * N + n], acc);
+    }
     out[(size_t)t * N + n] = from_f32<T>(acc);
   }
 }
@@ -545,6 +654,21 @@ GF_EXPORT int gf_moe_route(const float* logits, int T, int E, int top, int renor
   if (E > kMaxExperts || top > E || top > 32) return -3;
   return launch_kernel(moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, (cudaStream_t)stream,
                        logits, T, E, top, renorm, sigmoid, idx, wgt);
+}
+
+// See moe_route_grouped_kernel.
+GF_EXPORT int gf_moe_route_grouped(const float* logits, int ld, int T, int E, int identity, int top,
+                                   int groups, int keep, const float* correction, int gate_col,
+                                   int* idx, float* wgt, float* identity_w, float* gate,
+                                   void* stream) {
+  if (T <= 0) return 0;
+  if (E <= 0 || E > kMaxExperts || identity < 0 || identity > E || top < 1 || groups < 1 ||
+      E % groups || keep < 1 || keep > groups || top > E / groups * keep || ld < E ||
+      (gate && (gate_col < 0 || gate_col >= ld)))
+    return -3;
+  return launch_kernel(moe_route_grouped_kernel, dim3((T + 3) / 4), dim3(128), 0,
+                       (cudaStream_t)stream, logits, ld, T, E, identity, top, groups, keep,
+                       correction, gate_col, idx, wgt, identity_w, gate);
 }
 
 GF_EXPORT int gf_moe_plan(const int* idx, int P, int E, int tile_rows, int* offsets,
@@ -622,14 +746,15 @@ GF_EXPORT int gf_moe_gemm(const void* a, int lda, const void* w, int N, int K, c
 #undef GF_GO
 }
 
-GF_EXPORT int gf_moe_gather_rows(const void* x, int ldx, const int* pair_of_pos, int top, int P,
-                                 int K, void* xs, void* stream) {
+// placed: how many pairs have a place in the sorted order (offsets + E of the plan).
+GF_EXPORT int gf_moe_gather_rows(const void* x, int ldx, const int* pair_of_pos, const int* placed,
+                                 int top, int P, int K, void* xs, void* stream) {
   if (P <= 0) return 0;
   if (K % 8 || ldx % 8 || ((uintptr_t)x & 15) || ((uintptr_t)xs & 15)) return -3;
   const size_t want = ((size_t)P * (K / 8) + 255) / 256;
   const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
   return launch_kernel(moe_gather_rows_kernel, dim3(blocks), dim3(256), 0, (cudaStream_t)stream,
-                       (const bf*)x, ldx, pair_of_pos, top, P, K, (bf*)xs);
+                       (const bf*)x, ldx, pair_of_pos, placed, top, P, K, (bf*)xs);
 }
 
 GF_EXPORT int gf_moe_combine(const float* y, const int* pos_of_pair, const float* wgt, int T,

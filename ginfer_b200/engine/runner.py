@@ -266,15 +266,21 @@ class ModelRunner:
 
     def binder(self, dev: dict[str, torch.Tensor]):
         def bind(entry, block=False):
-            cid = entry.block_state if block else entry.cache
+            if isinstance(entry, int):                # a state by its number
+                return StateBinding(self.storage.state[entry], True)
+            if not block and isinstance(entry.cache, tuple):
+                return tuple(bind_one(c, entry.write_cache) for c in entry.cache)
+            return bind_one(entry.block_state if block else entry.cache,
+                            block or entry.write_cache)
+
+        def bind_one(cid, write):
             if self.storage.is_paged(cid):
                 g = self.storage.group_of(cid)
                 return PagedKVBinding(self.storage.pages_of(cid), dev[f"block_table{g}"],
                                       dev[f"slot_mapping{g}"], self.page_size,
-                                      self.groups[g].window, entry.write_cache,
-                                      self.groups[g].chunk)
+                                      self.groups[g].window, write, self.groups[g].chunk)
             if cid in self.storage.state:
-                return StateBinding(self.storage.state[cid], block or entry.write_cache)
+                return StateBinding(self.storage.state[cid], write)
             return None
         return bind
 

@@ -305,12 +305,13 @@ def mask_span(window: int = 0, chunk: int = 0) -> int:
 
 def paged_attention_simt(qkv, pages, block_table, seq_of_token, positions, nh, nkv, hd, scale,
                          window, page_size, vd=None, softcap: float = 0.0, slopes=None,
-                         sink: float | None = None):
+                         sink=None):
     """``window``: the mask as :func:`mask_span` gives it.  ``vd``: the values' head size where
     it is not the keys' (``pages`` is then a pair of tensors).  ``softcap`` > 0: scores pass
     ``cap * tanh(s / cap)``; ``slopes`` (fp32, a head): ``slope * (p - c)`` is taken off the score
     of the key at ``c`` for the query at ``p``, after the cap; ``sink``: ``exp(sink)`` is added to the
-    softmax's denominator (a score without a key and a value)."""
+    softmax's denominator (a score without a key and a value; a tensor: one a head)."""
+    from . import attention_bf16
     _cuda(qkv, pages[0], pages[1], block_table, seq_of_token, positions, slopes)
     assert slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == nh
                               and slopes.is_contiguous())
@@ -320,11 +321,11 @@ def paged_attention_simt(qkv, pages, block_table, seq_of_token, positions, nh, n
     f = _fn("attention_simt", "gf_paged_attention_simt",
             [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
              c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_float,
-             c_int, c_void_p])
+             c_void_p, c_int, c_void_p])
     rc = f(_p(qkv), qkv.stride(0), _p(pages[0]), _p(pages[1]), _p(block_table),
            block_table.stride(0), _p(seq_of_token), _p(positions), _p(out), T, nh, nkv, hd, vd,
            page_size, int(window), float(scale), float(softcap or 0.0), _p(slopes),
-           float("-inf") if sink is None else float(sink), _code(qkv.dtype), _stream())
+           *attention_bf16.sink_args(sink), _code(qkv.dtype), _stream())
     if rc == -3:
         raise ValueError(f"attention kernels take head sizes up to 256 and head counts that are "
                          f"a multiple of the kv head count; got head_dim={hd}, heads={nh}, "
@@ -343,7 +344,7 @@ def attention_fuses_rope(qkv: torch.Tensor, ctx, nh: int, nkv: int, hd: int) -> 
 def paged_attention(qkv: torch.Tensor, pages, block_table: torch.Tensor, ctx,
                     nh: int, nkv: int, hd: int, scale: float, window: int, page_size: int,
                     rope=None, vd: int | None = None, softcap: float = 0.0,
-                    slopes=None, sink: float | None = None) -> torch.Tensor:
+                    slopes=None, sink=None) -> torch.Tensor:
     """Attention of the step's queries (first ``nh * hd`` columns of ``qkv``) over the paged
     cache; returns ``[T, nh * hd]``.  Picks the kernel by dtype, head size and batch shape.
     ``rope = (table or None, rotary_dim, write)`` where :func:`attention_fuses_rope`: q and k are
@@ -444,4 +445,4 @@ def bmm_f32_out(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
 
 from .linear import GatedLinear, Linear, add_to  # noqa: E402,F401
 from . import prenorm  # noqa: E402,F401
-from . import depth, shift  # noqa: E402,F401
+from . import depth, hyper, rotary, shift  # noqa: E402,F401

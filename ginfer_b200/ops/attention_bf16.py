@@ -15,6 +15,16 @@ _scratch: dict = {}
 NO_SINK = float("-inf")
 
 
+def sink_args(sink):
+    """What the kernels are told of a sink: one score for all heads (``None``: none), or an fp32 tensor
+    with one a head -> ``(score, pointer)``."""
+    if torch.is_tensor(sink):
+        from . import _p
+        assert sink.dtype == torch.float32 and sink.dim() == 1 and sink.is_contiguous()
+        return NO_SINK, _p(sink)
+    return (NO_SINK if sink is None else float(sink)), None
+
+
 def supports(hd: int, nh: int, nkv: int) -> bool:
     return hd % 16 == 0 and 16 <= hd <= 256 and nh % nkv == 0
 
@@ -79,7 +89,7 @@ def _scratch_for(nbytes: int, device) -> torch.Tensor:
 def decode(qkv, pages, block_table, cu_seqlens_q, positions, B, nh, nkv, hd, scale, window,
            page_size, splits, out=None, scratch=None, through_scratch=False, rope=None,
            use_tma=True, stages=3, parts=1, softcap: float = 0.0, slopes=None,
-           sink: float | None = None):
+           sink=None):
     """Split-KV decode attention.  ``splits`` of 2, 4, 8 or 16 merge inside a thread-block cluster
     (no scratch memory) unless ``through_scratch``; any other number goes through scratch.
     ``rope = (table or None, rotary_dim, write)``: q and k arrive unrotated and the kernel
@@ -92,8 +102,8 @@ def decode(qkv, pages, block_table, cu_seqlens_q, positions, B, nh, nkv, hd, sca
     adds their results up (see :func:`decode_partition`).
     ``softcap`` > 0, ``slopes`` (fp32, a head): shaped scores as in ``ops.paged_attention_simt``;
     they take the kernel that loads its tiles with ``cp.async`` (no rotation inside it).
-    ``sink``: the score of a sink in the softmax's denominator (every kernel takes it; no rotation
-    inside it either)."""
+    ``sink``: the score of a sink in the softmax's denominator, a number or an fp32 tensor with one a
+    head (every kernel takes it; no rotation inside it either)."""
     from . import _fn, _ok, _p, _stream
     defines = (f"GF_HEAD_DIM={hd}",)
     is_shaped = bool(softcap) or slopes is not None
@@ -101,7 +111,8 @@ def decode(qkv, pages, block_table, cu_seqlens_q, positions, B, nh, nkv, hd, sca
         assert rope is None, "shaped scores and a rotation inside the kernel do not go together"
         use_tma = False
     assert rope is None or sink is None, "a sink and a rotation inside the kernel do not go together"
-    sink_score = NO_SINK if sink is None else float(sink)
+    assert not torch.is_tensor(sink) or sink.numel() == nh
+    sink_score, sinks = sink_args(sink)
     if out is None:
         out = torch.empty((qkv.shape[0], nh * hd), dtype=torch.bfloat16, device=qkv.device)
     if splits > 1 and scratch is None and (through_scratch or splits not in (2, 4, 8, 16)):
@@ -126,7 +137,7 @@ def decode(qkv, pages, block_table, cu_seqlens_q, positions, B, nh, nkv, hd, sca
         f = _fn("attention_bf16", "gf_attn_decode_tma",
                 [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                  c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p,
-                 c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_float], defines,
+                 c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_float, c_void_p], defines,
                 kernels=1)
         rc = f(_p(qkv), qkv.stride(0), _p(pages[0]), _p(pages[1]), pages.shape[1],
                _p(block_table), block_table.stride(0), _p(cu_seqlens_q), _p(positions), _p(out), B,
@@ -134,7 +145,7 @@ def decode(qkv, pages, block_table, cu_seqlens_q, positions, B, nh, nkv, hd, sca
                int(stages), _p(table),
                int(rot) if table is not None else 0, 1 if rope is not None else 0,
                int(bool(write)), _p(error_word(qkv.device)), _stream(), parts, _p(part_scratch),
-               sink_score)
+               sink_score, sinks)
         if rc == 0 and parts > 1:
             from . import _Counter
             _Counter.launches += 1                     # the kernel that adds the parts up
@@ -157,11 +168,11 @@ def decode(qkv, pages, block_table, cu_seqlens_q, positions, B, nh, nkv, hd, sca
         f = _fn("attention_bf16", "gf_attn_decode_shaped",
                 [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                  c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float,
-                 c_void_p, c_float, c_void_p], defines, kernels=1)
+                 c_void_p, c_float, c_void_p, c_void_p], defines, kernels=1)
         _ok(f(_p(qkv), qkv.stride(0), _p(pages[0]), _p(pages[1]), _p(block_table),
               block_table.stride(0), _p(cu_seqlens_q), _p(positions), _p(out), _p(scratch), B, nh,
               nkv, page_size, int(window), float(scale), int(splits), float(softcap or 0.0),
-              _p(slopes), sink_score, _stream()), "attn_decode_shaped")
+              _p(slopes), sink_score, sinks, _stream()), "attn_decode_shaped")
         return out
     f = _fn("attention_bf16", "gf_attn_decode",
             [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
@@ -175,7 +186,7 @@ def decode(qkv, pages, block_table, cu_seqlens_q, positions, B, nh, nkv, hd, sca
 
 def prefill(qkv, pages, block_table, cu_seqlens_q, kv_lens, B, max_q_len, nh, nkv, hd, scale,
             window, page_size, out=None, softcap: float = 0.0, slopes=None,
-            sink: float | None = None):
+            sink=None):
     from . import _fn, _ok, _p, _stream
     if out is None:
         out = torch.empty((qkv.shape[0], nh * hd), dtype=torch.bfloat16, device=qkv.device)
@@ -183,11 +194,11 @@ def prefill(qkv, pages, block_table, cu_seqlens_q, kv_lens, B, max_q_len, nh, nk
         f = _fn("attention_bf16", "gf_attn_prefill_shaped",
                 [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                  c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p,
-                 c_float, c_void_p], (f"GF_HEAD_DIM={hd}",))
+                 c_float, c_void_p, c_void_p], (f"GF_HEAD_DIM={hd}",))
         _ok(f(_p(qkv), qkv.stride(0), _p(pages[0]), _p(pages[1]), _p(block_table),
               block_table.stride(0), _p(cu_seqlens_q), _p(kv_lens), _p(out), B, int(max_q_len), nh,
               nkv, page_size, int(window), float(scale), float(softcap or 0.0), _p(slopes),
-              NO_SINK if sink is None else float(sink), _stream()), "attn_prefill_shaped")
+              *sink_args(sink), _stream()), "attn_prefill_shaped")
         return out
     f = _fn("attention_bf16", "gf_attn_prefill",
             [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
@@ -211,7 +222,7 @@ POLY_EXP_EVERY = int(os.environ.get("GINFER_B200_ATTN_POLY_EXP") or 0)
 
 def prefill_tc(qkv, pages, block_table, cu_seqlens_q, kv_lens, B, max_q_len, nh, nkv, hd, scale,
                window, page_size, trace=None, out=None, poly_exp_every: int | None = None,
-               softcap: float = 0.0, slopes=None, sink: float | None = None):
+               softcap: float = 0.0, slopes=None, sink=None):
     """Prefill attention on tcgen05 (``csrc/attention_tc.cu``); ``None`` if it cannot serve the
     shapes.  ``trace``: an int64 tensor of ``768 + 4 * CTAs`` slots that receives clock stamps of
     the first CTA's phases ([role 0 softmax (by tile), 1 MMA (by a stream's tile), 2 loader][32][8])
@@ -238,11 +249,11 @@ def prefill_tc(qkv, pages, block_table, cu_seqlens_q, kv_lens, B, max_q_len, nh,
         f = _fn("attention_tc", "gf_attn_prefill_tc_shaped",
                 [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                  c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-                 c_void_p, c_float, c_void_p, c_void_p, c_void_p], defines)
+                 c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p], defines)
         rc = f(_p(qkv), qkv.stride(0), _p(pages[0]), _p(pages[1]), pages.shape[1],
                _p(block_table), block_table.stride(0), _p(cu_seqlens_q), _p(kv_lens), _p(out), T,
                B, int(max_q_len), nh, nkv, page_size, int(window), float(scale),
-               float(softcap or 0.0), _p(slopes), NO_SINK if sink is None else float(sink),
+               float(softcap or 0.0), _p(slopes), *sink_args(sink),
                _p(_dev_state(qkv.device)["err"]), _p(trace), _stream())
     else:
         f = _fn("attention_tc", "gf_attn_prefill_tc",
@@ -269,7 +280,7 @@ def fuses_rope(qkv, ctx, hd: int, nh: int, nkv: int) -> bool:
 
 
 def try_run(qkv, pages, block_table, ctx, nh, nkv, hd, scale, window, page_size, rope=None,
-            softcap: float = 0.0, slopes=None, sink: float | None = None):
+            softcap: float = 0.0, slopes=None, sink=None):
     """Run a bf16 kernel if one takes this head size; ``None`` hands the work to the plain
     fp32-arithmetic kernel.  ``rope``: see :func:`decode` (only where :func:`fuses_rope`).
     ``window``: the mask as ``ops.mask_span`` gives it (negative: chunks)."""

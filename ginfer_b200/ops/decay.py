@@ -82,12 +82,14 @@ WIDE_MIN_TOKENS = 64
 
 
 def recurrence(q, k, v, g, state: torch.Tensor, ctx, H: int, G: int, D: int, Vd: int,
-               k_scale=None, skip=None) -> torch.Tensor:
+               k_scale=None, skip=None, normaliser: int | None = None):
     """Advance every request's state ``S [H, D, Vd]`` (first in its slot) over its tokens of this
     step: ``S <- diag(g_t) S + (c_t k_t) v_t^T``, ``o_t = S^T q_t + skip_h v_t``.  ``q``, ``k``:
     fp32 rows of ``G`` heads of ``D`` (views with a row stride are fine); ``v``: rows of ``H`` heads
     of ``Vd``; ``g``: rows of ``H * D`` decays, or of ``H`` (one a head); ``k_scale``: rows of
-    ``H`` factors ``c`` or ``None``; ``skip``: ``[H]`` or ``None``.  Returns ``o [T, H * Vd]``."""
+    ``H`` factors ``c`` or ``None``; ``skip``: ``[H]`` or ``None``.  Returns ``o [T, H * Vd]``.
+    ``normaliser``: where the slot's sums of keys ``n [H, D]`` start; they follow ``n <- diag(g_t) n +
+    c_t k_t`` and the result is ``(o, n_t . q_t [T, H])``."""
     _cuda(q, k, v, g, k_scale, skip, state)
     T = v.shape[0]
     for t in (q, k, v, g, k_scale):
@@ -97,43 +99,75 @@ def recurrence(q, k, v, g, state: torch.Tensor, ctx, H: int, G: int, D: int, Vd:
     assert g.shape[1] == H * gD and gD in (1, D)
     assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous()
     o = torch.empty((T, H * Vd), dtype=torch.float32, device=v.device)
+    o_n = None if normaliser is None else torch.empty((T, H), dtype=torch.float32, device=v.device)
     blocks = ctx.num_seqs * H * (-(-Vd // 32))
     wide = int(blocks < WIDE_BELOW_BLOCKS and ctx.max_q_len >= WIDE_MIN_TOKENS)
     f = _fn("decay_state", "gf_decay_recurrence",
             [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p,
              c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 5 +
-            [c_void_p, c_int, c_int, c_void_p])
+            [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p])
     rc = f(_p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(g), g.stride(0), gD,
            _p(k_scale), k_scale.stride(0) if k_scale is not None else 0, _p(skip), _p(state),
            state.stride(0), _p(ctx.cu_seqlens_q), _p(ctx.slot_ids), ctx.num_seqs, H, G, D, Vd,
-           _p(o), o.stride(0), wide, _stream())
+           _p(o), o.stride(0), wide, int(normaliser or 0), _p(o_n), H, _stream())
     if rc == -3:
         raise ValueError(f"the recurrence takes key sizes up to 256 and heads that are a multiple "
                          f"of the groups; got key size {D}, {H} heads, {G} groups")
     _ok(rc, "decay_recurrence")
-    return o
+    return o if o_n is None else (o, o_n)
+
+
+def memory_gates(proj: torch.Tensor, i_col: int, f_col: int, i_bias, f_bias, cap: float,
+                 state: torch.Tensor, m_off: int, ctx, H: int):
+    """Exponential gates of ``H`` heads from fp32 ``proj [T, ...]`` (input gates' columns from ``i_col``,
+    forget gates' from ``f_col``): ``i = cap tanh((z_i + b_i) / cap)``, ``f = log_sigmoid(cap
+    tanh((z_f + b_f) / cap))``.  The running maximum ``m_t = max(f_t + m_(t-1), i_t)`` is carried in
+    the slots (from ``m_off`` on; zero at a sequence's start).  Returns fp32 ``[T, H]`` each: decays
+    ``exp(f_t + m_(t-1) - m_t)``, factors ``exp(i_t - m_t)``, ``m_t``."""
+    _cuda(proj, i_bias, f_bias, state)
+    assert proj.dtype == torch.float32 and proj.dim() == 2 and proj.stride(1) == 1
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous()
+    for b in (i_bias, f_bias):
+        assert b.dtype == torch.float32 and b.numel() == H and b.is_contiguous()
+    out = torch.empty((3, proj.shape[0], H), dtype=torch.float32, device=proj.device)
+    f = _fn("decay_state", "gf_memory_gates",
+            [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int,
+             c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
+    _ok(f(_p(proj), proj.stride(0), int(i_col), int(f_col), _p(i_bias), _p(f_bias), float(cap),
+          _p(state), state.stride(0), int(m_off), _p(ctx.cu_seqlens_q), _p(ctx.slot_ids),
+          ctx.num_seqs, H, int(ctx.max_q_len), _p(out[0]), _p(out[1]), _p(out[2]),
+          int(ctx.max_q_len == 1), _stream()), "memory_gates")
+    return out[0], out[1], out[2]
 
 
 def gated_norm(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, group_size: int,
-               gate_first: bool, eps: float, dtype: torch.dtype, sigmoid_gate: bool = False
-               ) -> torch.Tensor:
+               gate_first: bool, eps: float, dtype: torch.dtype, sigmoid_gate: bool = False,
+               normaliser=None) -> torch.Tensor:
     """RMS norm of ``o [T, C]`` (fp32) in groups of ``group_size`` channels with a SiLU gate (a
     plain sigmoid with ``sigmoid_gate``):
     ``gate_first``: ``y = o silu(gate)``, then ``y / rms(y) * w``; else ``o / rms(o) * w *
-    silu(gate)``.  ``w`` has ``C`` weights, or ``group_size`` shared by the groups.  ``gate``:
+    silu(gate)``.  ``w`` has ``C`` weights, or ``group_size`` shared by the groups, or is
+    ``None``.  ``normaliser = (n [T, groups], m [T, groups], scale, floor)``: ``o`` is first multiplied by
+    ``scale / (max(|scale n|, exp(-m)) + floor)``, group by group.  ``gate``:
     ``[T, C]``, fp32 or the activation dtype, rows may be strided.  Returns ``[T, C]`` in
     ``dtype``."""
-    _cuda(o, gate, w)
+    _cuda(o, gate, w, *(normaliser or ())[:2])
     T, C = o.shape
     assert o.dtype == torch.float32 and o.is_contiguous() and C % group_size == 0
     assert gate.shape == (T, C) and gate.stride(1) == 1
-    assert w.dtype == torch.float32 and w.numel() in (C, group_size) and w.is_contiguous()
+    assert w is None or (w.dtype == torch.float32 and w.numel() in (C, group_size)
+                         and w.is_contiguous())
+    n, m, n_scale, floor = normaliser or (None, None, 1.0, 0.0)
+    for v in (n, m):
+        assert v is None or (v.dtype == torch.float32 and v.is_contiguous()
+                             and v.numel() == T * (C // group_size))
     out = torch.empty((T, C), dtype=dtype, device=o.device)
     f = _fn("decay_state", "gf_gated_norm",
             [c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_int,
-             c_int, c_int, c_int, c_void_p])
-    shared = int(w.numel() == group_size and C != group_size)
+             c_int, c_int, c_void_p, c_void_p, c_float, c_float, c_int, c_void_p])
+    shared = int(w is not None and w.numel() == group_size and C != group_size)
     _ok(f(_p(o), _p(gate), gate.stride(0), _code(gate.dtype), _p(w), shared, int(bool(gate_first)) | (2 if sigmoid_gate else 0),
-          float(eps), _p(out), T, C // group_size, int(group_size), _code(dtype), _stream()),
+          float(eps), _p(out), T, C // group_size, int(group_size), _p(n), _p(m), float(n_scale),
+          float(floor), _code(dtype), _stream()),
         "gated_norm")
     return out

@@ -76,8 +76,45 @@ def route(logits: torch.Tensor, top: int, renormalize: bool, score: str = "softm
     return idx, wgt
 
 
+def route_grouped(logits: torch.Tensor, experts: int, identity: int, top: int, correction=None,
+                  groups: int = 1, keep: int = 1, gate_col: int | None = None):
+    """fp32 rows ``[T, >= experts + identity]`` (``identity`` experts without matrices are the last of
+    the router's outputs) -> ``(experts [T, top] int32, weights [T, top], identity weights [T] or
+    None, gates [T] or None)``, fp32.  Scores: the softmax over all outputs.  Choice scores: with
+    ``correction`` (fp32, one an output) added.  With ``groups`` only outputs of the ``keep`` groups
+    (equal, of neighbours) with the largest best choice score can be chosen; the ``top`` with the
+    largest choice scores are, lowest index among equals; the weights are their scores.  A chosen
+    identity expert is ``-1`` with weight 0, its score counts in the identity weight.  ``gate_col``:
+    the column whose sigmoid is the token's gate."""
+    _cuda(logits, correction)
+    assert logits.dtype == torch.float32 and logits.dim() == 2 and logits.is_contiguous()
+    T, ld = logits.shape
+    E = experts + identity
+    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == E
+                                  and correction.is_contiguous())
+    dev = logits.device
+    idx = torch.empty((T, top), dtype=torch.int32, device=dev)
+    wgt = torch.empty((T, top), dtype=torch.float32, device=dev)
+    idw = torch.empty((T,), dtype=torch.float32, device=dev) if identity else None
+    gate = torch.empty((T,), dtype=torch.float32, device=dev) if gate_col is not None else None
+    f = _fn("moe", "gf_moe_route_grouped",
+            [c_void_p] + [c_int] * 7 + [c_void_p, c_int] + [c_void_p] * 5)
+    rc = f(_p(logits), ld, T, E, int(identity), int(top), int(groups), int(keep), _p(correction),
+           int(gate_col or 0), _p(idx), _p(wgt), _p(idw), _p(gate), _stream())
+    if rc == -3:
+        raise ValueError(f"the router kernel takes up to {MAX_EXPERTS} outputs in equal groups and no "
+                         f"more choices than the kept groups hold; got {E} outputs, {groups} groups, "
+                         f"{keep} kept, {top} choices")
+    _ok(rc, "moe_route_grouped")
+    return idx, wgt, idw, gate
+
+
+MAX_EXPERTS = 256
+
+
 class Plan:
-    """Where every (token, choice) pair sits once the pairs are sorted by expert."""
+    """Where every (token, choice) pair sits once the pairs are sorted by expert; a pair of expert
+    ``-1`` sits nowhere (position ``-1``)."""
 
     def __init__(self, idx: torch.Tensor, num_experts: int, tensor_cores=False):
         T, top = idx.shape
@@ -133,10 +170,10 @@ def gather_rows(x: torch.Tensor, plan: Plan) -> torch.Tensor:
     """The tokens' rows in the order of the sorted pairs, ``[P, K]``."""
     K = x.shape[1]
     xs = torch.empty((plan.pairs, K), dtype=x.dtype, device=x.device)
-    f = _fn("moe", "gf_moe_gather_rows", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p,
-                                          c_void_p])
-    _ok(f(_p(x), x.stride(0), _p(plan.pair_of_pos), plan.top, plan.pairs, K, _p(xs), _stream()),
-        "moe_gather_rows")
+    f = _fn("moe", "gf_moe_gather_rows", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
+                                          c_void_p, c_void_p])
+    _ok(f(_p(x), x.stride(0), _p(plan.pair_of_pos), _p(plan.offsets[plan.num_experts:]), plan.top,
+          plan.pairs, K, _p(xs), _stream()), "moe_gather_rows")
     return xs
 
 

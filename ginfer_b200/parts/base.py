@@ -167,6 +167,36 @@ class PairSum:
 
 
 @dataclass
+class TermSum:
+    """The output of a sublayer that is a sum, not added up yet: dense ``terms`` ``(tensor [T, H],
+    constant, factors [T] fp32 or None)`` (the first one fp32, a second one fp32 or the activation
+    dtype) and a routed feed-forward's ``pairs``.  A kernel that adds the output to the stream can form
+    the sum itself; anything else calls :meth:`materialize`."""
+    terms: list
+    pairs: PairSum | None = None
+
+    def kernel_args(self) -> dict:
+        p = self.pairs
+        return dict(terms=self.terms,
+                    pairs=None if p is None else (p.rows, p.pos_of_pair, p.weights, p.top))
+
+    def materialize(self) -> torch.Tensor:
+        from ..ops import hyper
+        some = self.terms[0][0] if self.terms else self.pairs.rows
+        one = torch.ones(1, dtype=torch.float32, device=some.device)
+        return hyper.update(None, 1, torch.float32, out_w=one, **self.kernel_args())[0][:, 0]
+
+
+@dataclass
+class MixedInput:
+    """What the first sublayer of a run reads, where the model carries several residual streams: the
+    norm of their sum with the fp32 ``weights [streams]``.  It takes the place of the plain norm where
+    another block prepares a run's input (``then``)."""
+    norm: "Norm"
+    weights: torch.Tensor
+
+
+@dataclass
 class ShiftedInput:
     """What the first sublayer of a run reads, where that is a norm of the stream shifted towards
     the token before: ``n_t + (n_(t-1) - n_t) * weight`` with ``n = norm(x)`` and ``weight`` fp32
@@ -239,8 +269,19 @@ class Mixer(Part):
     takes_lazy_norm = False
     adds_residual = False
 
-    def cache_spec(self) -> PagedKVSpec | StateSpec | None:
+    def cache_spec(self) -> PagedKVSpec | StateSpec | tuple | None:
+        """What the mixer keeps; a tuple for a mixer made of several, which then gets a tuple of
+        bindings."""
         return None
+
+    # A mixer that sets this takes the keyword ``defer_terms`` and may then return a :class:`TermSum`
+    # instead of its output.
+    defers_terms = False
+
+    # A mixer whose work starts with ONE product of its input, left in 32-bit, may offer it to a mixer
+    # that runs several on the same input: ``input_matrix(tensors)`` (rows a multiple of 8, called
+    # before ``load``, which then makes no product of its own) and ``from_projection(p, ctx, cache)``.
+    shares_input_product = False
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache) -> torch.Tensor:
         raise NotImplementedError
@@ -249,6 +290,9 @@ class Mixer(Part):
 class FeedForward(Part):
     takes_lazy_norm = False
     adds_residual = False
+    # A feed-forward that sets this takes the keyword ``defer_terms`` and may then return a
+    # :class:`TermSum` instead of its output.
+    defers_terms = False
     # A feed-forward that sets this takes the keyword ``defer_sum`` and may then return a
     # :class:`PairSum` instead of its output.
     can_defer_sum = False
@@ -265,8 +309,9 @@ class Block(Part):
     # A block that sets this takes the keyword ``then``: the norm that will consume its output
     # (the next run's first norm), so that its last product can prepare that norm's input.
     takes_next_norm = False
-    # ``then`` may be a :class:`ShiftedInput`
+    # ``then`` may be a :class:`ShiftedInput`, a :class:`MixedInput`
     prepares_shifted_input = False
+    prepares_mixed_input = False
 
     def forward(self, x: torch.Tensor, delta: torch.Tensor | None, ctx: StepContext, cache
                 ) -> tuple[torch.Tensor, torch.Tensor | None]:
@@ -281,7 +326,8 @@ class Block(Part):
     def state_spec(self) -> StateSpec | None:
         return None
 
-    def first_input(self, own_state: StateBinding | None) -> "Norm | ShiftedInput | None":
+    def first_input(self, own_state: StateBinding | None
+                    ) -> "Norm | ShiftedInput | MixedInput | None":
         """What another block may prepare for this one, given the binding of its own state."""
         return self.first_norm()
 
@@ -307,6 +353,11 @@ class StreamInput(Part):
 
 
 class Embedding(Part):
+    # An embedding that depends on earlier tokens of the sequence says what it keeps of them, and its
+    # ``forward`` takes the keyword ``own_state`` (a :class:`StateBinding`).
+    def state_spec(self) -> StateSpec | None:
+        return None
+
     def forward(self, token_ids: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         raise NotImplementedError
 

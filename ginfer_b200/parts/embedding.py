@@ -10,7 +10,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
-from .base import Embedding, Head, TensorSpec, register_part
+from .base import Embedding, Head, StateSpec, TensorSpec, register_part
 
 
 class TokenEmbedding(Embedding):
@@ -74,6 +74,37 @@ class PositionedEmbedding(Embedding):
         return x
 
 
+class BigramEmbedding(Embedding):
+    """``x[t] = E[token] * scale + P[row]`` with a table ``P [buckets + 1, hidden]`` over pairs of
+    neighbouring tokens: ``row = (token before * mul_prev + token * mul_cur) mod buckets``, the last row
+    for a sequence's first token.  The fp32 residual stream.  The token before a step's first one is
+    per-request state."""
+
+    def __init__(self, vocab_size: int, hidden_size: int, buckets: int, mul_prev: int, mul_cur: int,
+                 scale: float = 1.0, name: str = "embed", table_name: str = "bigram"):
+        self.vocab_size, self.hidden_size = int(vocab_size), int(hidden_size)
+        self.buckets, self.mul_prev, self.mul_cur = int(buckets), int(mul_prev), int(mul_cur)
+        if self.buckets < 1 or self.mul_prev < 0 or self.mul_cur < 0:
+            raise ValueError("a pair table has at least one bucket and no negative multiplier")
+        self.scale, self.name, self.table_name = float(scale), name, table_name
+        self.weight: torch.Tensor | None = None
+        self.table: torch.Tensor | None = None
+
+    def tensor_specs(self):
+        return [TensorSpec(self.name, (self.vocab_size, self.hidden_size), "embedding"),
+                TensorSpec(self.table_name, (self.buckets + 1, self.hidden_size), "embedding")]
+
+    def load(self, tensors, dtype, device):
+        self.weight, self.table = tensors[self.name], tensors[self.table_name]
+
+    def state_spec(self):
+        return StateSpec((1,), torch.int32)
+
+    def forward(self, token_ids, ctx, own_state):
+        return ops.hyper.bigram_embedding(token_ids, self.weight, self.scale, self.table, self.buckets,
+                                          self.mul_prev, self.mul_cur, own_state.state, ctx)
+
+
 class LinearHead(Head):
     """``tied_to`` names the tensor of another part (the embedding) to share; otherwise the head
     has a matrix ``name`` of its own.  ``softcap``: the logits pass ``cap * tanh(logits / cap)``
@@ -103,4 +134,5 @@ class LinearHead(Head):
 
 register_part("embedding", "token", TokenEmbedding)
 register_part("embedding", "token_positions", PositionedEmbedding)
+register_part("embedding", "token_bigram", BigramEmbedding)
 register_part("head", "linear", LinearHead)

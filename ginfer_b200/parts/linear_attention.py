@@ -16,7 +16,8 @@ import torch
 
 from .. import ops
 from ..ops import decay
-from .base import Mixer, StateSpec, TensorSpec, register_mixer
+from .base import Mixer, StateSpec, TensorSpec, make_part, register_mixer
+from .plan import PartSpec
 
 
 class GatedLinearAttention(Mixer):
@@ -141,3 +142,88 @@ class DecayLinearAttention(Mixer):
 
 
 register_mixer("decay_linear_attention", DecayLinearAttention)
+
+
+def joined_rows(parts: list[torch.Tensor], multiple: int = 8) -> torch.Tensor:
+    """Matrices on top of each other, with zero rows up to a multiple of ``multiple`` rows."""
+    n = sum(x.shape[0] for x in parts)
+    pad = -n % multiple
+    if pad:
+        parts = parts + [torch.zeros((pad, parts[0].shape[1]), dtype=parts[0].dtype,
+                                     device=parts[0].device)]
+    return torch.cat(parts, dim=0)
+
+
+class Retention(Mixer):
+    """Linear attention with one fixed decay a head and rotated queries and keys.  ``q = W_q h``, ``k =
+    W_k h`` (``H`` heads of ``D``), ``v = W_v h`` (``H`` heads of ``Vd``); q and k are rotated by the
+    position encoding (``None``: not), k times ``D^-1/2``; per head ``S_t = a_n S_(t-1) + k_t v_t^T``,
+    ``o_t = S_t^T q_t``.  Each head's ``o`` is RMS-normed without a weight, times ``silu(W_g h)``,
+    projected by ``W_o``.
+
+    State per request (one fp32 row of a slot): ``S [H, D, Vd]``, zero at the start.  One product gives
+    q | k | v | g in 32-bit; rotation, recurrence, norm and gate are fp32 arithmetic in both paths."""
+
+    shares_input_product = True
+
+    def __init__(self, hidden_size: int, num_heads: int, key_dim: int, v_dim: int, decays,
+                 position: PartSpec | None = None, norm_eps: float = 1e-6, prefix: str = "mix"):
+        self.hidden_size, self.H = int(hidden_size), int(num_heads)
+        self.D, self.Vd = int(key_dim), int(v_dim)
+        self.decays = [float(a) for a in decays]
+        if len(self.decays) != self.H:
+            raise ValueError(f"{len(self.decays)} decays for {self.H} heads")
+        if self.D > decay.MAX_KEY_SIZE:
+            raise ValueError(f"a key size of {self.D} is over the recurrence kernel's "
+                             f"{decay.MAX_KEY_SIZE}")
+        self.position = make_part("position", position) if position is not None else None
+        if self.position is not None:
+            if not hasattr(self.position, "frequencies") or self.position.mult != 1.0:
+                raise ValueError("this mixer rotates channel pairs by plain frequencies (position kind "
+                                 "'pair_rotary')")
+            if self.position.dims > self.D:
+                raise ValueError(f"{self.position.dims} rotated channels do not fit a head of {self.D}")
+        self.eps = float(norm_eps)
+        self.prefix = prefix + "." if prefix else ""
+        self.first = None
+
+    def _n(self, name):
+        return self.prefix + name
+
+    def tensor_specs(self):
+        W, HD, HV = self.hidden_size, self.H * self.D, self.H * self.Vd
+        return [TensorSpec(self._n("q"), (HD, W)), TensorSpec(self._n("k"), (HD, W)),
+                TensorSpec(self._n("v"), (HV, W)), TensorSpec(self._n("g"), (HV, W)),
+                TensorSpec(self._n("o"), (W, HV))]
+
+    def input_matrix(self, tensors):
+        return joined_rows([tensors[self._n(k)] for k in ("q", "k", "v", "g")])
+
+    def load(self, tensors, dtype, device, own_product: bool = True):
+        if own_product:
+            self.first = ops.Linear(self.input_matrix(tensors), None, out_dtype=torch.float32)
+        self.out = ops.Linear(tensors[self._n("o")], None, out_dtype=torch.float32)
+        self.decay_row = torch.tensor(self.decays, dtype=torch.float32, device=device)[None, :]
+        if self.position is not None:
+            self.position.load(tensors, dtype, device)
+
+    def cache_spec(self):
+        return StateSpec((self.H * self.D * self.Vd,), torch.float32)
+
+    def forward(self, x, ctx, cache):
+        return self.from_projection(self.first(x), ctx, cache)
+
+    def from_projection(self, p, ctx, cache):
+        H, D, Vd = self.H, self.D, self.Vd
+        HD, HV = H * D, H * Vd                              # p: fp32 [T, q | k | v | g (| pad)]
+        pos = self.position
+        ops.rotary.heads_(p, H, H, D, 0, HD, pos.frequencies() if pos is not None else None,
+                          pos.interleaved if pos is not None else False, D ** -0.5, ctx)
+        g = self.decay_row.expand(p.shape[0], H)            # every token's decays: the constants
+        o = decay.recurrence(p[:, :HD], p[:, HD:2 * HD], p[:, 2 * HD:2 * HD + HV], g, cache.state, ctx,
+                             H, H, D, Vd)
+        y = decay.gated_norm(o, p[:, 2 * HD + HV:2 * HD + 2 * HV], None, Vd, False, self.eps, ctx.dtype)
+        return self.out(y)
+
+
+register_mixer("retention", Retention)

@@ -9,7 +9,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import StepContext, Summed, TensorSpec, make_part
+from .base import MixedInput, StepContext, Summed, TensorSpec, make_part
 from .plan import ModelPlan
 
 
@@ -77,10 +77,22 @@ class DecoderModel:
     # ------------------------------------------------------------------ caches
     def cache_specs(self) -> dict[int, object]:
         """Cache id -> spec, taken from the layer whose run writes that cache."""
+        def of_mixer(e) -> tuple:
+            spec = self.blocks[e.layer].mixer.cache_spec()
+            specs = spec if isinstance(spec, tuple) else (spec,)
+            if len(specs) != len(e.caches()):
+                raise ValueError(f"a run of layer {e.layer} names {len(e.caches())} caches; its mixer "
+                                 f"keeps {len(specs)}")
+            return specs
         out: dict[int, object] = {}
+        own = self.embedding.state_spec()
+        if (own is None) != (self.plan.embedding_state is None):
+            raise ValueError("the plan and the embedding disagree on whether it keeps a state")
+        if own is not None:
+            out[self.plan.embedding_state] = own
         for e in self.plan.run:
             if e.write_cache:
-                out[e.cache] = self.blocks[e.layer].mixer.cache_spec()
+                out.update(zip(e.caches(), of_mixer(e)))
             own = self.blocks[e.layer].state_spec()
             if (own is None) != (e.block_state is None):
                 raise ValueError(f"a run of layer {e.layer} and its block disagree on whether the "
@@ -89,26 +101,33 @@ class DecoderModel:
                 out[e.block_state] = own
         for e in self.plan.run:
             if not e.write_cache:
-                mine = self.blocks[e.layer].mixer.cache_spec()
-                if mine != out[e.cache]:
-                    raise ValueError(f"layer {e.layer} cannot read cache {e.cache}: it holds "
-                                     f"{out[e.cache]} but the layer expects {mine}")
+                for c, mine in zip(e.caches(), of_mixer(e)):
+                    if mine != out[c]:
+                        raise ValueError(f"layer {e.layer} cannot read cache {c}: it holds "
+                                         f"{out[c]} but the layer expects {mine}")
         return out
 
-    def _next_input(self, entry, own_state):
-        """What the block before may prepare for ``entry``'s run: nothing where its block's own
-        state is needed for that and not at hand."""
+    def _next_input(self, blk, entry, own_state):
+        """What ``blk`` may prepare for ``entry``'s run behind it: nothing where that run's block needs
+        its own state for it and the state is not at hand, or where ``blk`` does not know how."""
         if entry.block_state is not None and own_state is None:
             return None
-        return self.blocks[entry.layer].first_input(own_state)
+        first = self.blocks[entry.layer].first_input(own_state)
+        if isinstance(first, MixedInput) and not blk.prepares_mixed_input:
+            return None
+        return first
 
     # ------------------------------------------------------------------ one step
     def forward(self, ctx: StepContext, bind_cache) -> torch.Tensor:
         """Run the step's tokens; ``bind_cache(run_entry)`` gives the cache binding of a run,
-        ``bind_cache(run_entry, block=True)`` that of its block's own state.
+        ``bind_cache(run_entry, block=True)`` that of its block's own state, ``bind_cache(id)`` that
+        of a state by its number.
         Returns fp32 logits ``[R, vocab]`` at ``ctx.logit_rows``."""
         delta = None
-        x = self.embedding.forward(ctx.token_ids, ctx)
+        own = {}
+        if self.plan.embedding_state is not None:
+            own["own_state"] = bind_cache(self.plan.embedding_state)
+        x = self.embedding.forward(ctx.token_ids, ctx, **own)
         embedded = x
         run = self.plan.run
         for i, e in enumerate(run):
@@ -127,7 +146,7 @@ class DecoderModel:
                 if n.block_state is not None and blk.prepares_shifted_input:
                     own = bind_cache(n, block=True)
                 x, delta = blk.forward(x, delta, ctx, bind_cache(e),
-                                       then=self._next_input(n, own), **kw)
+                                       then=self._next_input(blk, n, own), **kw)
             else:
                 x, delta = blk.forward(x, delta, ctx, bind_cache(e), **kw)
         if ctx.logit_rows.numel() == 0:

@@ -37,16 +37,20 @@ class LayerSpec:
 class RunEntry:
     """One run of a layer.  ``layer`` indexes :attr:`ModelPlan.layers` (a layer may be named
     twice).  ``cache`` names the cache this run uses: by default a cache of its own; a run with
-    ``write_cache=False`` only reads the cache another run has written earlier in the step.
+    ``write_cache=False`` only reads the cache another run has written earlier in the step.  A mixer
+    made of several names a cache for each, in their order (a tuple).
     ``enter = (i, n)``: before this run the stream passes through
     :attr:`ModelPlan.stream_inputs` ``[i]`` as its entry number ``n`` (the start of a pass of a
     loop, say).  ``block_state`` names the per-request state of the layer's block itself, beside
     its mixer's cache (for blocks that keep one)."""
     layer: int
-    cache: int
+    cache: int | tuple[int, ...]
     write_cache: bool = True
     enter: tuple[int, int] | None = None
     block_state: int | None = None
+
+    def caches(self) -> tuple[int, ...]:
+        return self.cache if isinstance(self.cache, tuple) else (self.cache,)
 
 
 @dataclass(frozen=True)
@@ -61,6 +65,7 @@ class ModelPlan:
     head: PartSpec
     eos_token_ids: tuple[int, ...] = ()
     stream_inputs: tuple[PartSpec, ...] = ()   # parts that runs enter through (RunEntry.enter)
+    embedding_state: int | None = None   # the per-request state of the embedding, if it keeps one
     ignored_tensors: tuple[str, ...] = ()     # regular expressions of tensor names to pass over
 
     def validate(self) -> None:
@@ -72,19 +77,22 @@ class ModelPlan:
             if e.enter is not None and not (0 <= e.enter[0] < len(self.stream_inputs)):
                 raise ValueError(f"run[{pos}] enters through stream input {e.enter[0]}, but "
                                  f"there are {len(self.stream_inputs)}")
-            if e.write_cache:
-                if e.cache in writers:
-                    raise ValueError(f"run[{pos}] and run[{writers[e.cache]}] both write cache "
-                                     f"{e.cache}")
-                writers[e.cache] = pos
+            for c in e.caches() if e.write_cache else ():
+                if c in writers:
+                    raise ValueError(f"run[{pos}] and run[{writers[c]}] both write cache {c}")
+                writers[c] = pos
             if e.block_state is not None:
                 if e.block_state in writers:
                     raise ValueError(f"run[{pos}] keeps its block's state as {e.block_state}, "
                                      f"which run[{writers[e.block_state]}] writes")
                 writers[e.block_state] = pos
         for pos, e in enumerate(self.run):
-            if not e.write_cache and (e.cache not in writers or writers[e.cache] > pos):
-                raise ValueError(f"run[{pos}] reads cache {e.cache} before any run writes it")
+            for c in () if e.write_cache else e.caches():
+                if c not in writers or writers[c] > pos:
+                    raise ValueError(f"run[{pos}] reads cache {c} before any run writes it")
+        if self.embedding_state is not None and self.embedding_state in writers:
+            raise ValueError(f"the embedding keeps its state as {self.embedding_state}, which "
+                             f"run[{writers[self.embedding_state]}] writes")
 
 
 def sequential_run(num_layers: int) -> tuple[RunEntry, ...]:

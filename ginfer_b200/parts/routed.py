@@ -17,7 +17,8 @@ import torch
 
 from .. import ops
 from ..ops import moe
-from .base import FeedForward, PairSum, TensorSpec, register_feed_forward
+from .base import FeedForward, PairSum, TensorSpec, TermSum, register_feed_forward
+from .linear_attention import joined_rows
 
 
 class RoutedGLU(FeedForward):
@@ -127,3 +128,82 @@ class RoutedExperts(FeedForward):
 
 
 register_feed_forward("routed_experts", RoutedExperts)
+
+
+class GroupRoutedGLU(RoutedGLU):
+    """A :class:`RoutedGLU` chosen in groups.  Router scores ``s``: softmax over ALL outputs, ``experts``
+    of them with matrices and then ``identity`` experts without (their output is their input).  Choice
+    scores are ``s`` plus ``<prefix>.correction``; the outputs form ``groups`` equal groups of neighbours,
+    the ``keep_groups`` with the largest best choice score stay, and of their outputs the ``top_k`` with
+    the largest choice scores are chosen; the weights are their ``s``.  ``shared_size`` > 0: a shared
+    expert of the same form runs for every token, times ``sigmoid(<prefix>.shared.sg h)``.
+
+    The shared gate's logit is one more row of the router's product.  The output is left as a sum
+    (:class:`TermSum`): the chosen experts' rows, the input times the identity weights, and the shared
+    expert's output times its gate."""
+
+    can_defer_sum = False
+    defers_terms = True
+
+    def __init__(self, hidden_size: int, intermediate_size: int, num_experts: int, top_k: int,
+                 identity: int = 0, groups: int = 1, keep_groups: int = 1, shared_size: int = 0,
+                 limit: float = float("inf"), alpha: float = 1.0, up_shift: float = 0.0,
+                 prefix: str = "mlp"):
+        super().__init__(hidden_size, intermediate_size, limit, num_experts,
+                         min(int(top_k), int(num_experts)), False, alpha, up_shift, prefix)
+        self.top, self.identity = int(top_k), int(identity)
+        self.groups, self.keep, self.shared_size = int(groups), int(keep_groups), int(shared_size)
+        outputs = self.E + self.identity
+        if outputs > moe.MAX_EXPERTS:
+            raise ValueError(f"{outputs} router outputs are over the kernel's {moe.MAX_EXPERTS}")
+        if self.groups < 1 or outputs % self.groups or not (1 <= self.keep <= self.groups):
+            raise ValueError(f"{outputs} router outputs do not form {groups} equal groups of which "
+                             f"{keep_groups} stay")
+        if not (0 < self.top <= outputs // self.groups * self.keep):
+            raise ValueError(f"{self.top} choices among the {outputs // self.groups * self.keep} outputs "
+                             "of the kept groups")
+
+    def tensor_specs(self):
+        h, f, p = self.hidden_size, self.shared_size, self.prefix
+        outputs = self.E + self.identity
+        out = [s for s in super().tensor_specs() if s.name != p + "router"]
+        out += [TensorSpec(p + "router", (outputs, h)), TensorSpec(p + "correction", (outputs,), "f32")]
+        if f:
+            out += [TensorSpec(p + "shared.gate", (f, h)), TensorSpec(p + "shared.up", (f, h)),
+                    TensorSpec(p + "shared.down", (h, f)), TensorSpec(p + "shared.sg", (1, h))]
+        return out
+
+    def load(self, tensors, dtype, device):
+        super().load(tensors, dtype, device)
+        p = self.prefix
+        rows = [tensors[p + "router"]] + ([tensors[p + "shared.sg"]] if self.shared_size else [])
+        self.router = ops.Linear(joined_rows(rows), None, out_dtype=torch.float32)
+        self.correction = tensors[p + "correction"].float().contiguous()
+        self.shared = self.shared_down = None
+        if self.shared_size:
+            self.shared = ops.GatedLinear(tensors[p + "shared.gate"], tensors[p + "shared.up"],
+                                          clamped=(self.limit, self.alpha, self.up_shift))
+            self.shared_down = ops.Linear(tensors[p + "shared.down"], None, out_dtype=torch.float32)
+
+    def forward(self, x, ctx, defer_terms: bool = False):
+        T = x.shape[0]
+        idx, wgt, idw, gate = moe.route_grouped(
+            self.router(x), self.E, self.identity, self.top, self.correction, self.groups, self.keep,
+            self.E + self.identity if self.shared_size else None)
+        plan = moe.Plan(idx, self.E, moe.kernel_for(
+            x, T * self.top, (self.hidden_size, self.intermediate_size),
+            (self.intermediate_size, self.hidden_size)))
+        y = moe.grouped_glu(x, self.w_gate_up, plan, self.limit, self.alpha, self.up_shift,
+                            act=self.act)
+        rows = moe.grouped_down(y, self.w_down, plan)
+        terms = []
+        if self.shared is not None:
+            terms.append((self.shared_down(self.shared(x)), 1.0, gate))
+        if idw is not None:
+            terms.append((x, 1.0, idw))
+        out = TermSum(terms, PairSum(rows, plan.pos_of_pair, wgt, self.top,
+                                     lambda: moe.combine(rows, plan, wgt, T)))
+        return out if defer_terms else out.materialize()
+
+
+register_feed_forward("group_routed_glu", GroupRoutedGLU)
