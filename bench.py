@@ -375,6 +375,35 @@ def lasizen_config(width, heads, kv_heads, dim, window, ff, layers, vocab=32768)
                        for i in range(layers)]}
 
 
+def daburax_config(width, heads, kv_heads, dim, experts, identity, top, expert_ff, layers, vocab=32768):
+    """Layers in turns of four on four streams, each with a mixture of experts (chosen in four groups,
+    two kept, some identities, one shared expert): retention, retention, attention with sinks beside a
+    matrix memory, retention."""
+    retention = {"type": "retention", "mixer": {
+        "heads": heads, "dim": dim, "vdim": dim, "rot": {"base": 10000.0, "dims": dim},
+        "decay": [1.0 - 2.0 ** (-5.0 - 4.0 * n / heads) for n in range(heads)]}}
+    parallel = {"type": "parallel", "mixer": {
+        "left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                 "rot": {"base": 10000.0, "dims": dim // 2, "scaling": {"factor": 4.0}}},
+        "right": {"heads": heads, "dim": dim, "vdim": dim, "gate_cap": 15.0},
+        "left_scale": 1.0, "right_scale": 0.5}}
+    mlp = {"kind": "moe", "expert": {"ff": expert_ff}, "shared": {"ff": expert_ff},
+           "router": {"experts": experts - identity, "identity": identity, "top": top,
+                      "groups": {"count": 4, "keep": 2}}}
+    return {"architecture": "Daburax", "width": width, "vocab": vocab, "norm": {"eps": 1e-6},
+            "streams": 4, "residual_mult": 0.5, "torch_dtype": "bfloat16",
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 32749, "mul_prev": 257, "mul_cur": 31}},
+            "layers": [dict(parallel if i % 4 == 2 else retention, mlp=mlp) for i in range(layers)]}
+
+
+DABURAX_SIZES = {
+    # width, heads, kv heads, dim, router outputs, identity experts among them, top, expert ff (the
+    # shared expert has the same)
+    "s": (1024, 8, 2, 64, 16, 2, 2, 704),
+    "m": (2048, 16, 4, 128, 32, 4, 4, 1408),
+}
+
+
 LASIZEN_SIZES = {
     # width, heads, kv heads, dim, window, two-matrix ff (Vilepel beside it: a three-matrix ff of two
     # thirds of that)
@@ -450,6 +479,18 @@ def design_configs(design: str, name: str, layers: int) -> dict:
             "vilepel": vilepel_config(width, heads, dim, dim // 2, dim, width // 4, window,
                                       2 * ff // 3, 1, 1, 1, layers, routed=False),
         }
+    if design == "daburax":
+        # beside it the closest design the engine has, Pimidra (linear attention with decays,
+        # grouped-query attention over every earlier key, routed feed-forwards of the same experts, an
+        # fp32 stream), at the same width, heads, head size, router and expert sizes and layer count
+        width, heads, kv, dim, experts, identity, top, eff = DABURAX_SIZES[name]
+        beside = pimidra_config(width, heads, kv, dim, CONTEXT, 2 * eff, experts, top, eff, heads, dim,
+                                dim, 4)
+        gla, moe = beside["layers"][3], beside["layers"][2]["mlp"]
+        beside["layers"] = [dict(beside["layers"][2] if i % 4 == 2 else gla, mlp=moe)
+                            for i in range(layers)]
+        return {"daburax": daburax_config(width, heads, kv, dim, experts, identity, top, eff, layers),
+                "pimidra": beside}
     if design == "pimidra":
         # beside it the closest design the engine has, Vilepel (attention with a bounded reach and a
         # recurrent mixer in turns, dense and routed feed-forwards, an fp32 stream), at the same
@@ -479,11 +520,15 @@ def run_design(args) -> int:
     out = {"design": args.design,
            "beside": ("vilepel at equal width, heads, head size, feed-forward sizes, reach and "
                       "layers" if args.design in ("pimidra", "bapivik", "lasizen") else
+                      "pimidra (linear attention with decays and attention in the same turns, all "
+                      "feed-forwards routed) at equal width, heads, head size, router and expert "
+                      "sizes and layers" if args.design == "daburax" else
                       "qwen2 at equal width, heads, feed-forward arithmetic and layer runs"),
            "dtype": "bfloat16", "data": "synthetic", "sizes": {}}
     layers = args.layers or 8
     sizes = {"zolapel": ZOLAPEL_SIZES, "pimidra": PIMIDRA_SIZES,
-             "bapivik": BAPIVIK_SIZES, "lasizen": LASIZEN_SIZES}.get(args.design, DESIGN_SIZES)
+             "bapivik": BAPIVIK_SIZES, "lasizen": LASIZEN_SIZES,
+             "daburax": DABURAX_SIZES}.get(args.design, DESIGN_SIZES)
     for name in (args.size.split(",") if args.size else sorted(sizes)):
         cfgs = design_configs(args.design, name, layers)
         width = sizes[name][0]
@@ -512,7 +557,7 @@ def run_design(args) -> int:
 MICRO = ("gemm_gateup_m8", "gemm_down_m8", "gemm_lmhead_m8", "gemm_gateup_m2048", "gemm_qkv_m2048",
          "attn_decode_b8",
          "attn_decode_b64", "attn_decode_b1_ctx32768", "prefill_2layers", "bapivik_prefill_4layers",
-         "lasizen_prefill_2layers")
+         "lasizen_prefill_2layers", "daburax_prefill_4layers")
 
 
 def run_micro(name: str) -> int:
@@ -602,7 +647,7 @@ def run_micro(name: str) -> int:
         torch.cuda.synchronize()
         print(json.dumps({"micro": name, "tokens": PREFILL_TOKENS}))
         return 0
-    if name in ("bapivik_prefill_4layers", "lasizen_prefill_2layers"):
+    if name in ("bapivik_prefill_4layers", "lasizen_prefill_2layers", "daburax_prefill_4layers"):
         # one turn of the design's layers at size m, a 2,048-token prompt three times
         from ginfer_b200.engine import StepEntry
         from ginfer_b200.engine.llm import Engine
@@ -832,7 +877,8 @@ def main() -> int:
                     help="tokens a step of the long prompt in --scenario longctx (default 2,048)")
     ap.add_argument("--scenario", choices=SCENARIOS, default=None,
                     help="run a serving workload through the entry point instead of the benchmark")
-    ap.add_argument("--design", choices=["vilepel", "zolapel", "pimidra", "bapivik", "lasizen"], default=None,
+    ap.add_argument("--design", choices=["vilepel", "zolapel", "pimidra", "bapivik", "lasizen", "daburax"],
+                    default=None,
                     help="measure another design beside Qwen2 at equal size instead of the benchmark")
     ap.add_argument("--size", default=None, help="with --design: sizes to run, e.g. s,m")
     args = ap.parse_args()

@@ -144,6 +144,11 @@ __device__ __forceinline__ void pdl_trigger() {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
 }
 
+// An index that a kernel shortly before this one wrote, read from L2.  A kernel that was launched while
+// that one still ran may share its SM with kernels that read the same memory when it held something
+// else (a recycled buffer), and what they left in L1 must not be taken for an index.
+__device__ __forceinline__ int fresh_index(const int* p) { return __ldcg(p); }
+
 inline int& pdl_flag() {
   static int enabled = 1;
   return enabled;

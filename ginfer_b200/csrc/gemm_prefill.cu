@@ -238,7 +238,7 @@ gemm_prefill_kernel(const __grid_constant__ CUtensorMap tmap_x,
   const uint32_t tmem = *tmem_slot;
   if (GROUPED) {
     pdl_wait();                                // the list of row tiles comes from a kernel ahead
-    m_tiles = grp.num_tiles[0];
+    m_tiles = fresh_index(grp.num_tiles);
   }
   const int ntiles = m_tiles * n_tiles;
 
@@ -251,8 +251,8 @@ gemm_prefill_kernel(const __grid_constant__ CUtensorMap tmap_x,
         int n0 = (tile / m_tiles) * PN + (PAIR ? (int)rank * (PN / 2) : 0);
         int m0 = (tile % m_tiles) * TM + (int)rank * PM;
         if (GROUPED) {                                 // the group's matrix; the tile's first row
-          n0 += grp.tile_expert[tile % m_tiles] * N;
-          m0 = grp.tile_row0[tile % m_tiles];
+          n0 += fresh_index(grp.tile_expert + tile % m_tiles) * N;
+          m0 = fresh_index(grp.tile_row0 + tile % m_tiles);
         }
         for (int kb = 0; kb < nkb; ++kb, ++it) {
           const int s = it % NST;
@@ -339,11 +339,11 @@ gemm_prefill_kernel(const __grid_constant__ CUtensorMap tmap_x,
       int m = (tile % m_tiles) * TM + (int)rank * PM + q * 32 + lane;
       float row_scale = 1.f;
       if (GROUPED) {                                   // rows past the group's end are not stored
-        const int mt = tile % m_tiles, row0 = grp.tile_row0[mt];
-        const int end = grp.offsets[grp.tile_expert[mt] + 1];
+        const int mt = tile % m_tiles, row0 = fresh_index(grp.tile_row0 + mt);
+        const int end = fresh_index(grp.offsets + fresh_index(grp.tile_expert + mt) + 1);
         m = row0 + q * 32 + lane;
         if (m >= end) m = M;
-        if (EPI == PEPI_RELU2 && grp.row_w && m < M) row_scale = grp.row_w[grp.pair_of_pos[m]];
+        if (EPI == PEPI_RELU2 && grp.row_w && m < M) row_scale = grp.row_w[fresh_index(grp.pair_of_pos + m)];
       }
       const float* bias_t = bias_s + buf * PN + half * (PN / 2);     // of this thread's columns
       if (EPI != PEPI_GATED && EPI != PEPI_RELU2 && bias) {

@@ -109,8 +109,8 @@ hyper_update_vec_kernel(const HyperArgs a) {
       float y[4] = {0.f, 0.f, 0.f, 0.f};
       if (a.pair_rows) {
         for (int k = 0; k < a.top; ++k) {
-          const int p = a.pair_pos[src * a.top + k];
-          if (p < 0) continue;
+          const int p = fresh_index(a.pair_pos + src * a.top + k);
+          if ((unsigned)p >= gridDim.x * (unsigned)a.top) continue;        // no row
           const float pw = a.pair_w ? a.pair_w[src * a.top + k] : 1.f;
           float v[4];
           Quad<float>::load(a.pair_rows + (size_t)p * W + j, v);
@@ -171,8 +171,8 @@ __global__ void hyper_update_kernel(const HyperArgs a) {
     float y = 0.f, u = 0.f;
     if (a.pair_rows) {
       for (int k = 0; k < a.top; ++k) {
-        const int p = a.pair_pos[src * a.top + k];
-        if (p >= 0)
+        const int p = fresh_index(a.pair_pos + src * a.top + k);
+        if ((unsigned)p < gridDim.x * (unsigned)a.top)
           y = fmaf(a.pair_w ? a.pair_w[src * a.top + k] : 1.f, a.pair_rows[(size_t)p * W + j], y);
       }
     }

@@ -208,7 +208,7 @@ moe_plan_kernel(const int* __restrict__ idx, int P, int E, int tile_rows,
   int mine_in_run = 0;
   for (int p0 = p_lo; p0 < p_hi; p0 += 32) {
     const int p = p0 + lane;
-    const int g = p < p_hi ? idx[p] : -1;
+    const int g = p < p_hi ? fresh_index(idx + p) : -1;
     if (g >= 0 && g != e) atomicAdd(&count[g], 1);
     mine_in_run += __popc(__ballot_sync(0xffffffffu, g == e));
   }
@@ -241,7 +241,8 @@ moe_plan_kernel(const int* __restrict__ idx, int P, int E, int tile_rows,
   for (int w = 0; w < warp; ++w) at += run_count[w];
   for (int p0 = p_lo; p0 < p_hi; p0 += 32) {
     const int p = p0 + lane;
-    const bool mine = p < p_hi && idx[p] == e;
+    const int g = p < p_hi ? fresh_index(idx + p) : e + 1;
+    const bool mine = g == e;
     const unsigned m = __ballot_sync(0xffffffffu, mine);
     if (mine) {
       const int pos = at + __popc(m & ((1u << lane) - 1));
@@ -249,7 +250,7 @@ moe_plan_kernel(const int* __restrict__ idx, int P, int E, int tile_rows,
       pair_of_pos[pos] = p;
     }
     at += __popc(m);
-    if (e == 0 && p < p_hi && idx[p] < 0) pos_of_pair[p] = -1;
+    if (e == 0 && g < 0) pos_of_pair[p] = -1;
   }
 }
 
@@ -278,14 +279,14 @@ moe_gemm_kernel(const T* __restrict__ a, int lda, const T* __restrict__ w, int N
   __shared__ int src_row[kBM];
   pdl_trigger();
   pdl_wait();
-  if ((int)blockIdx.x >= num_tiles[0]) return;
-  const int e = tile_expert[blockIdx.x], row0 = tile_row0[blockIdx.x];
-  const int rows = min(kBM, offsets[e + 1] - row0);
+  if ((int)blockIdx.x >= fresh_index(num_tiles)) return;
+  const int e = fresh_index(tile_expert + blockIdx.x), row0 = fresh_index(tile_row0 + blockIdx.x);
+  const int rows = min(kBM, fresh_index(offsets + e + 1) - row0);
   const int n0 = blockIdx.y * kBN;
   const T* we = w + (size_t)e * N * K;
   if (threadIdx.x < kBM) {
     const int s = row0 + threadIdx.x;
-    src_row[threadIdx.x] = threadIdx.x < rows ? (FIRST ? pair_of_pos[s] / top : s) : -1;
+    src_row[threadIdx.x] = threadIdx.x < rows ? (FIRST ? fresh_index(pair_of_pos + s) / top : s) : -1;
   }
   __syncthreads();
   const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;    // rows 2 ty, 2 ty + 1; cols 4 tx ..
@@ -394,14 +395,14 @@ moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_bfl
   __shared__ int src_row[kTM];
   pdl_trigger();
   pdl_wait();
-  if ((int)blockIdx.x >= num_tiles[0]) return;
-  const int e = tile_expert[blockIdx.x], row0 = tile_row0[blockIdx.x];
-  const int rows = min(kTM, offsets[e + 1] - row0);
+  if ((int)blockIdx.x >= fresh_index(num_tiles)) return;
+  const int e = fresh_index(tile_expert + blockIdx.x), row0 = fresh_index(tile_row0 + blockIdx.x);
+  const int rows = min(kTM, fresh_index(offsets + e + 1) - row0);
   const int n0 = blockIdx.y * kTN;
   const __nv_bfloat16* we = w + (size_t)e * N * K;
   if (threadIdx.x < kTM) {
     const int s = row0 + threadIdx.x;
-    src_row[threadIdx.x] = threadIdx.x < rows ? (FIRST ? pair_of_pos[s] / top : s) : -1;
+    src_row[threadIdx.x] = threadIdx.x < rows ? (FIRST ? fresh_index(pair_of_pos + s) / top : s) : -1;
   }
   __syncthreads();
   const int nk = (K + kTK - 1) / kTK;
@@ -519,13 +520,13 @@ moe_gemv_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_bfloat1
   extern __shared__ __align__(16) __nv_bfloat16 xrows[];           // [kFewRows][K]
   pdl_trigger();
   pdl_wait();
-  if ((int)blockIdx.x >= num_tiles[0]) return;
-  const int e = tile_expert[blockIdx.x], row0 = tile_row0[blockIdx.x];
-  const int rows = min(kFewRows, offsets[e + 1] - row0);
+  if ((int)blockIdx.x >= fresh_index(num_tiles)) return;
+  const int e = fresh_index(tile_expert + blockIdx.x), row0 = fresh_index(tile_row0 + blockIdx.x);
+  const int rows = min(kFewRows, fresh_index(offsets + e + 1) - row0);
   const int k8 = K >> 3;
   for (int i = threadIdx.x; i < rows * k8; i += blockDim.x) {
     const int r = i / k8, c = (i - r * k8) * 8;
-    const int src = MODE != 0 ? pair_of_pos[row0 + r] / top : row0 + r;
+    const int src = MODE != 0 ? fresh_index(pair_of_pos + row0 + r) / top : row0 + r;
     *reinterpret_cast<uint4*>(xrows + (size_t)r * K + c) =
         *reinterpret_cast<const uint4*>(a + (size_t)src * lda + c);
   }
@@ -608,12 +609,12 @@ __global__ void moe_gather_rows_kernel(const __nv_bfloat16* __restrict__ x, int 
   pdl_trigger();
   pdl_wait();
   const int k8 = K >> 3;
-  P = min(P, *placed);                              // pairs that have a place
+  P = min(P, fresh_index(placed));                  // pairs that have a place
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < (size_t)P * k8;
        i += (size_t)gridDim.x * blockDim.x) {
     const size_t s = i / k8;
     const int c = (int)(i - s * k8) * 8;
-    const size_t src = (size_t)(pair_of_pos[s] / top) * ldx + c;
+    const size_t src = (size_t)(fresh_index(pair_of_pos + s) / top) * ldx + c;
     *reinterpret_cast<uint4*>(xs + s * K + c) = *reinterpret_cast<const uint4*>(x + src);
   }
 }
@@ -628,7 +629,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
   for (int n = threadIdx.x; n < N; n += blockDim.x) {
     float acc = 0.f;
     for (int k = 0; k < top; ++k) {
-      const int p = pos_of_pair[(size_t)t * top + k];
+      const int p = fresh_index(pos_of_pair + (size_t)t * top + k);
       if (p >= 0) acc = fmaf(wgt ? wgt[(size_t)t * top + k] : 1.f, y[(size_t)p * N + n], acc);
     }
     out[(size_t)t * N + n] = from_f32<T>(acc);

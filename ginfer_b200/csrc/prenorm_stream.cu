@@ -49,7 +49,7 @@ __global__ void stream_update_kernel(const float* __restrict__ x, const int* __r
         v = 0.f;
         for (int k = 0; k < top; ++k) {
           const size_t pr = (src / H) * top + k;
-          v = fmaf(pair_w ? pair_w[pr] : 1.f, to_f32(y[(size_t)pos_of_pair[pr] * H + j]), v);
+          v = fmaf(pair_w ? pair_w[pr] : 1.f, to_f32(y[(size_t)fresh_index(pos_of_pair + pr) * H + j]), v);
         }
       } else {
         v = to_f32(y[src + j]);
@@ -126,7 +126,7 @@ __global__ void stream_update_vec_kernel(const float* __restrict__ x, const int*
             const size_t pr = (src / H) * top + k;
             const float pw = pair_w ? pair_w[pr] : 1.f;
             float t[4];
-            Quad<Y>::load(y + (size_t)pos_of_pair[pr] * H + 4 * q, t);
+            Quad<Y>::load(y + (size_t)fresh_index(pos_of_pair + pr) * H + 4 * q, t);
 #pragma unroll
             for (int i = 0; i < 4; ++i) v[u][i] = fmaf(pw, t[i], v[u][i]);
           }

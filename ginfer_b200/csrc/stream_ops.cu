@@ -109,7 +109,7 @@ __device__ __forceinline__ float post_y(const Y* __restrict__ y, const int* __re
   if (pos == nullptr) return to_f32(y[(size_t)r * H + j]);
   float a = 0.f;
   for (int k = 0; k < top; ++k) {
-    const float v = to_f32(y[(size_t)pos[r * top + k] * H + j]);
+    const float v = to_f32(y[(size_t)fresh_index(pos + r * top + k) * H + j]);
     a = wgt != nullptr ? fmaf(wgt[r * top + k], v, a) : a + v;
   }
   return a;
@@ -173,7 +173,7 @@ __global__ void postnorm_vec_kernel(const float* __restrict__ x, const Y* __rest
         for (int i = 0; i < 4; ++i) yv[i] = 0.f;
         for (int k = 0; k < top; ++k) {
           float pv[4];
-          Quad<Y>::load(y + (size_t)pos[r * top + k] * H + 4 * q, pv);
+          Quad<Y>::load(y + (size_t)fresh_index(pos + r * top + k) * H + 4 * q, pv);
           const float w = wgt != nullptr ? wgt[r * top + k] : 1.f;
 #pragma unroll
           for (int i = 0; i < 4; ++i) yv[i] = wgt != nullptr ? fmaf(w, pv[i], yv[i]) : yv[i] + pv[i];
