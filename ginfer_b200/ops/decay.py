@@ -7,7 +7,7 @@ from ctypes import c_float, c_int, c_void_p
 
 import torch
 
-from . import _code, _cuda, _fn, _ok, _p, _stream
+from . import _code, _cuda, _fn, _ok, _p, _stream, load_library
 
 
 def ssd_prepare(proj: torch.Tensor, conv_col: int, dt_col: int, conv_w: torch.Tensor,
@@ -81,6 +81,35 @@ WIDE_BELOW_BLOCKS = 96
 WIDE_MIN_TOKENS = 64
 
 
+# Portions of at least this many tokens with one decay a head run a chunk of tokens at a time
+# (``csrc/decay_chunk.cu``).
+CHUNK_MIN_TOKENS = 64
+
+
+def _chunked(q, k, v, g, state, ctx, first: int, H, G, D, Vd, k_scale, skip, normaliser, o, o_n) -> bool:
+    """The requests from number ``first`` on, a chunk of tokens at a time; ``False`` if not served."""
+    if D > 128 or D % 4 or Vd % 4:
+        return False
+    if not _chunk_tokens:
+        _chunk_tokens.append(int(load_library("decay_chunk").gf_decay_chunk_tokens()))
+    chunks = sum(-(-n // _chunk_tokens[0]) for n in ctx.q_lens_host[first:])
+    scratch = torch.empty(chunks * H * (D * Vd + D + 1), dtype=torch.float32, device=v.device)
+    f = _fn("decay_chunk", "gf_decay_chunked",
+            [c_void_p, c_int] * 5 + [c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 6 +
+            [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p], kernels=3)
+    rc = f(_p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(g), g.stride(0), _p(k_scale),
+           k_scale.stride(0) if k_scale is not None else 0, _p(skip), _p(state), state.stride(0),
+           _p(ctx.cu_seqlens_q[first:]), _p(ctx.slot_ids[first:]), ctx.num_seqs - first, chunks, H, G, D,
+           Vd, _p(o), o.stride(0), int(normaliser or 0), _p(o_n), H, _p(scratch), _stream())
+    if rc == -6:
+        return False
+    _ok(rc, "decay_chunked")
+    return True
+
+
+_chunk_tokens: list = []
+
+
 def recurrence(q, k, v, g, state: torch.Tensor, ctx, H: int, G: int, D: int, Vd: int,
                k_scale=None, skip=None, normaliser: int | None = None):
     """Advance every request's state ``S [H, D, Vd]`` (first in its slot) over its tokens of this
@@ -100,15 +129,27 @@ def recurrence(q, k, v, g, state: torch.Tensor, ctx, H: int, G: int, D: int, Vd:
     assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous()
     o = torch.empty((T, H * Vd), dtype=torch.float32, device=v.device)
     o_n = None if normaliser is None else torch.empty((T, H), dtype=torch.float32, device=v.device)
-    blocks = ctx.num_seqs * H * (-(-Vd // 32))
-    wide = int(blocks < WIDE_BELOW_BLOCKS and ctx.max_q_len >= WIDE_MIN_TOKENS)
+    # long portions with one decay a head go a chunk at a time; single tokens in front of them (as the
+    # scheduler orders a mixed step) token by token
+    seqs, q_lens = ctx.num_seqs, getattr(ctx, "q_lens_host", ())
+    if gD == 1 and ctx.max_q_len >= CHUNK_MIN_TOKENS and len(q_lens) == seqs:
+        singles = 0
+        while q_lens[singles] == 1:
+            singles += 1
+        if _chunked(q, k, v, g, state, ctx, singles, H, G, D, Vd, k_scale, skip, normaliser, o, o_n):
+            if not singles:
+                return o if o_n is None else (o, o_n)
+            seqs = singles
+    blocks = seqs * H * (-(-Vd // 32))
+    wide = int(blocks < WIDE_BELOW_BLOCKS and seqs == ctx.num_seqs
+               and ctx.max_q_len >= WIDE_MIN_TOKENS)
     f = _fn("decay_state", "gf_decay_recurrence",
             [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p,
              c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 5 +
             [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p])
     rc = f(_p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(g), g.stride(0), gD,
            _p(k_scale), k_scale.stride(0) if k_scale is not None else 0, _p(skip), _p(state),
-           state.stride(0), _p(ctx.cu_seqlens_q), _p(ctx.slot_ids), ctx.num_seqs, H, G, D, Vd,
+           state.stride(0), _p(ctx.cu_seqlens_q), _p(ctx.slot_ids), seqs, H, G, D, Vd,
            _p(o), o.stride(0), wide, int(normaliser or 0), _p(o_n), H, _stream())
     if rc == -3:
         raise ValueError(f"the recurrence takes key sizes up to 256 and heads that are a multiple "

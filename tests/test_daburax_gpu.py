@@ -703,3 +703,50 @@ def test_attention_with_a_sink_a_head(hd, nh, nkv, page):
                 y = attention_bf16.decode(args[0], args[1], args[2], args[3].cu_seqlens_q, args[3].positions,
                                           len(ids), nh, nkv, hd, scale, 0, page, 8, parts=2, sink=sinks.cuda())
                 close(y, want, 2e-2)
+
+
+@pytest.mark.parametrize("H, G, D, Vd", [(3, 3, 32, 64), (4, 2, 20, 36), (2, 1, 128, 132), (2, 2, 64, 200),
+                                         (1, 1, 100, 8), (6, 3, 4, 4)])
+def test_a_chunk_of_tokens_at_a_time(monkeypatch, H, G, D, Vd):
+    """Long portions in chunks against token by token and against the equations, in one batch with short
+    portions and single tokens in front and behind, from states that are not zero; keys shared by groups of
+    heads, step factors, a skip, a normaliser; decays of zero, of one and of 1e-30."""
+    from ginfer_b200.ops import decay
+    g = torch.Generator().manual_seed(D * Vd)
+    lens, slots = [1, 1, 130, 5, 64, 1, 257], [6, 0, 3, 1, 7, 2, 4]
+    T = sum(lens)
+    n_off = H * D * Vd
+    q, k = torch.randn(T, G * D, generator=g), torch.randn(T, G * D, generator=g) * D ** -0.5
+    v, c = torch.randn(T, H * Vd, generator=g), torch.rand(T, H, generator=g)
+    decays = 1.0 - torch.rand(T, H, generator=g) ** 4
+    decays[::17], decays[5::31], decays[3::29] = 1.0, 0.0, 1e-30
+    skip = torch.randn(H, generator=g)
+    start = torch.randn(8, n_off + H * D + 3, generator=g)
+    ctx = packed(lens, slots)
+    got = {}
+    for name, limit in (("chunks", 64), ("tokens", 1 << 30)):
+        monkeypatch.setattr(decay, "CHUNK_MIN_TOKENS", limit)
+        a, b = start.cuda(), start.cuda()
+        args = [t.cuda() for t in (q, k, v, decays)]
+        plain_o = decay.recurrence(*args, a, ctx, H, G, D, Vd, k_scale=c.cuda(), skip=skip.cuda())
+        o, nq = decay.recurrence(*args, b, ctx, H, G, D, Vd, normaliser=n_off)
+        got[name] = [t.double().cpu() for t in (plain_o, a, o, nq, b)]
+    for x, y in zip(got["chunks"], got["tokens"]):
+        assert float((x - y).abs().max()) <= 2e-5 * float(y.abs().max())
+    # against the equations: the request of 130 tokens
+    at, n, s = sum(lens[:2]), lens[2], slots[2]
+    for h in range(H):
+        S = start[s, h * D * Vd:(h + 1) * D * Vd].double().view(D, Vd)
+        z = start[s, n_off + h * D:n_off + (h + 1) * D].double()
+        for t in range(at, at + n):
+            kk = k[t, (h // (H // G)) * D:][:D].double()
+            qq = q[t, (h // (H // G)) * D:][:D].double()
+            S = decays[t, h].double() * S + torch.outer(kk, v[t, h * Vd:(h + 1) * Vd].double())
+            z = decays[t, h].double() * z + kk
+            close(got["chunks"][2][t, h * Vd:(h + 1) * Vd], S.T @ qq, 2e-4)
+            close(got["chunks"][3][t, h], z @ qq, 2e-4)
+        close(got["chunks"][4][s, h * D * Vd:(h + 1) * D * Vd].view(D, Vd), S, 2e-4)
+        close(got["chunks"][4][s, n_off + h * D:n_off + (h + 1) * D], z, 2e-4)
+    # slots that no request of the step has, and what lies behind the states, stay as they were
+    assert torch.equal(got["chunks"][4][5], start[5].double())
+    assert torch.equal(got["chunks"][4][:, n_off + H * D:], start[:, n_off + H * D:].double())
