@@ -192,7 +192,7 @@ __global__ void silu_f32_vec_kernel(const __nv_bfloat16* __restrict__ proj, int 
 // A block a (head, request): a thread a token at a time, blockDim tokens together by a scan over the
 // maps m -> max(m + a, b), which compose to the same form.  Only m's own value depends on the order of
 // the sums; the factors are formed from the m that are written, so they fit together exactly.
-constexpr int kGateThreads = 256;
+constexpr int kGateThreads = 1024;
 __global__ void __launch_bounds__(kGateThreads)
 memory_gates_kernel(const float* __restrict__ proj, int ld, int i_col, int f_col,
                     const float* __restrict__ i_bias, const float* __restrict__ f_bias, float cap,

@@ -89,6 +89,8 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int T, int E,
 // index among equals).  idx: the expert, or -1 for an identity one; wgt: its s (0 for an identity one);
 // identity_w[t]: the sum of the identity ones' s (null: not wanted).  gate[t] = sigmoid(row[gate_col])
 // (null: no gate).
+// SLOTS: router outputs a lane.
+template <int SLOTS>
 __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int ld, int T, int E,
                                          int identity, int top, int groups, int keep,
                                          const float* __restrict__ correction, int gate_col,
@@ -103,10 +105,10 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int l
   pdl_wait();
   if (t >= T) return;                                         // (warps are independent)
   const float* row = logits + (size_t)t * ld;
-  float s[kRouteSlots], c[kRouteSlots];
+  float s[SLOTS], c[SLOTS];
   float mx = -INFINITY;
 #pragma unroll
-  for (int i = 0; i < kRouteSlots; ++i) {
+  for (int i = 0; i < SLOTS; ++i) {
     const int e = lane + 32 * i;
     s[i] = e < E ? row[e] : -INFINITY;
     mx = fmaxf(mx, s[i]);
@@ -114,13 +116,13 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int l
   mx = warp_max(mx);
   float sum = 0.f;
 #pragma unroll
-  for (int i = 0; i < kRouteSlots; ++i) {
+  for (int i = 0; i < SLOTS; ++i) {
     s[i] = expf(s[i] - mx);                                   // 0 past the last expert
     sum += s[i];
   }
   sum = warp_sum(sum);
 #pragma unroll
-  for (int i = 0; i < kRouteSlots; ++i) {
+  for (int i = 0; i < SLOTS; ++i) {
     const int e = lane + 32 * i;
     s[i] = s[i] / sum;
     c[i] = e < E ? s[i] + (correction ? correction[e] : 0.f) : -INFINITY;
@@ -131,7 +133,7 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int l
     for (int g = 0; g < groups; ++g) {
       float best = -INFINITY;
 #pragma unroll
-      for (int i = 0; i < kRouteSlots; ++i) {
+      for (int i = 0; i < SLOTS; ++i) {
         const int e = lane + 32 * i;
         if (e >= g * gs && e < (g + 1) * gs) best = fmaxf(best, c[i]);
       }
@@ -141,7 +143,7 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int l
     __syncwarp();
     // a group stays if fewer than `keep` groups come before it (larger, or equal with a lower index)
 #pragma unroll
-    for (int i = 0; i < kRouteSlots; ++i) {
+    for (int i = 0; i < SLOTS; ++i) {
       const int e = lane + 32 * i;
       if (e >= E) continue;
       const int g = e / gs;
@@ -156,7 +158,7 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int l
     float best = -INFINITY;
     int be = 0x7fffffff;
 #pragma unroll
-    for (int i = 0; i < kRouteSlots; ++i)
+    for (int i = 0; i < SLOTS; ++i)
       if (c[i] > best) best = c[i], be = lane + 32 * i;       // ascending e: lowest index wins
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
@@ -166,7 +168,7 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int l
     }
     float w = 0.f;
 #pragma unroll
-    for (int i = 0; i < kRouteSlots; ++i)
+    for (int i = 0; i < SLOTS; ++i)
       if (lane + 32 * i == be) w = s[i], c[i] = -INFINITY;
     w = __shfl_sync(0xffffffffu, w, be & 31);
     const bool none = be >= E0;                               // an identity expert (or none is left)
@@ -192,23 +194,28 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int l
 // earlier pairs of the same expert, whatever the grid.
 constexpr int kPlanThreads = 256, kPlanWarps = kPlanThreads / 32;
 __global__ void __launch_bounds__(kPlanThreads)
-moe_plan_kernel(const int* __restrict__ idx, int P, int E, int tile_rows,
+moe_plan_kernel(const int* __restrict__ idx, int P, int E, int tile_rows, int stage,
                 int* __restrict__ offsets, int* __restrict__ pos_of_pair,
                 int* __restrict__ pair_of_pos, int* __restrict__ tile_expert,
                 int* __restrict__ tile_row0, int* __restrict__ num_tiles) {
   __shared__ int count[kMaxExperts], run_count[kPlanWarps], base[2];
+  extern __shared__ int held[];                    // the pairs' experts, if they fit
   const int e = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_trigger();
   pdl_wait();
   for (int i = threadIdx.x; i < E; i += blockDim.x) count[i] = 0;
+  if (stage)
+#pragma unroll 8
+    for (int p = threadIdx.x; p < P; p += blockDim.x) held[p] = fresh_index(idx + p);
   __syncthreads();
+  auto expert_of = [&](int p) { return stage ? held[p] : fresh_index(idx + p); };
   // this block's expert by ballots over the warps' runs; the others by shared atomics
   const int run = (((P + kPlanWarps - 1) / kPlanWarps) + 31) & ~31;
   const int p_lo = warp * run, p_hi = min(P, p_lo + run);
   int mine_in_run = 0;
   for (int p0 = p_lo; p0 < p_hi; p0 += 32) {
     const int p = p0 + lane;
-    const int g = p < p_hi ? fresh_index(idx + p) : -1;
+    const int g = p < p_hi ? expert_of(p) : -1;
     if (g >= 0 && g != e) atomicAdd(&count[g], 1);
     mine_in_run += __popc(__ballot_sync(0xffffffffu, g == e));
   }
@@ -241,7 +248,7 @@ moe_plan_kernel(const int* __restrict__ idx, int P, int E, int tile_rows,
   for (int w = 0; w < warp; ++w) at += run_count[w];
   for (int p0 = p_lo; p0 < p_hi; p0 += 32) {
     const int p = p0 + lane;
-    const int g = p < p_hi ? fresh_index(idx + p) : e + 1;
+    const int g = p < p_hi ? expert_of(p) : e + 1;
     const bool mine = g == e;
     const unsigned m = __ballot_sync(0xffffffffu, mine);
     if (mine) {
@@ -667,9 +674,14 @@ GF_EXPORT int gf_moe_route_grouped(const float* logits, int ld, int T, int E, in
       E % groups || keep < 1 || keep > groups || top > E / groups * keep || ld < E ||
       (gate && (gate_col < 0 || gate_col >= ld)))
     return -3;
-  return launch_kernel(moe_route_grouped_kernel, dim3((T + 3) / 4), dim3(128), 0,
-                       (cudaStream_t)stream, logits, ld, T, E, identity, top, groups, keep,
-                       correction, gate_col, idx, wgt, identity_w, gate);
+#define GF_GO(SLOTS)                                                                              \
+  return launch_kernel(moe_route_grouped_kernel<SLOTS>, dim3((T + 3) / 4), dim3(128), 0,          \
+                       (cudaStream_t)stream, logits, ld, T, E, identity, top, groups, keep,       \
+                       correction, gate_col, idx, wgt, identity_w, gate)
+  if (E <= 32) GF_GO(1);
+  if (E <= 64) GF_GO(2);
+  GF_GO(kRouteSlots);
+#undef GF_GO
 }
 
 GF_EXPORT int gf_moe_plan(const int* idx, int P, int E, int tile_rows, int* offsets,
@@ -677,8 +689,10 @@ GF_EXPORT int gf_moe_plan(const int* idx, int P, int E, int tile_rows, int* offs
                           int* num_tiles, void* stream) {
   if (P <= 0) return 0;
   if (E > kMaxExperts || tile_rows <= 0) return -3;
-  return launch_kernel(moe_plan_kernel, dim3(E), dim3(kPlanThreads), 0, (cudaStream_t)stream, idx,
-                       P, E, tile_rows, offsets, pos_of_pair, pair_of_pos, tile_expert, tile_row0,
+  const size_t held = (size_t)P * sizeof(int);     // staged where it fits without asking for more
+  const int stage = held <= 40 * 1024;
+  return launch_kernel(moe_plan_kernel, dim3(E), dim3(kPlanThreads), stage ? held : 0,
+                       (cudaStream_t)stream, idx, P, E, tile_rows, stage, offsets, pos_of_pair, pair_of_pos, tile_expert, tile_row0,
                        num_tiles);
 }
 
