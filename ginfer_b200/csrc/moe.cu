@@ -88,13 +88,14 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int T, int E,
 // stay (lowest index among equals).  Of their experts the `top` with the largest c are chosen (lowest
 // index among equals).  idx: the expert, or -1 for an identity one; wgt: its s (0 for an identity one);
 // identity_w[t]: the sum of the identity ones' s (null: not wanted).  gate[t] = sigmoid(row[gate_col])
-// (null: no gate).
+// (null: no gate).  always > 0: every token has that many more pairs behind its choices, of the experts
+// E - identity, E - identity + 1, ..., with its gate as weight (rows of idx and wgt are top + always long).
 // SLOTS: router outputs a lane.
 template <int SLOTS>
 __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int ld, int T, int E,
                                          int identity, int top, int groups, int keep,
                                          const float* __restrict__ correction, int gate_col,
-                                         int* __restrict__ idx, float* __restrict__ wgt,
+                                         int always, int* __restrict__ idx, float* __restrict__ wgt,
                                          float* __restrict__ identity_w,
                                          float* __restrict__ gate) {
   constexpr int kW = 4;                                       // warps a block
@@ -152,7 +153,7 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int l
       if (ahead >= keep) c[i] = -INFINITY;
     }
   }
-  const int E0 = E - identity;
+  const int E0 = E - identity, ldk = top + always;
   float id_sum = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
@@ -174,13 +175,18 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int l
     const bool none = be >= E0;                               // an identity expert (or none is left)
     if (none) id_sum += w;
     if (lane == 0) {
-      idx[(size_t)t * top + k] = none ? -1 : be;
-      wgt[(size_t)t * top + k] = none ? 0.f : w;
+      idx[(size_t)t * ldk + k] = none ? -1 : be;
+      wgt[(size_t)t * ldk + k] = none ? 0.f : w;
     }
   }
-  if (lane == 0) {
-    if (identity_w) identity_w[t] = id_sum;
-    if (gate) gate[t] = 1.f / (1.f + expf(-row[gate_col]));
+  if (lane == 0 && identity_w) identity_w[t] = id_sum;
+  if (gate_col >= 0) {
+    const float gt = 1.f / (1.f + expf(-row[gate_col]));
+    if (lane == 0 && gate) gate[t] = gt;
+    if (lane < always) {
+      idx[(size_t)t * ldk + top + lane] = E0 + lane;
+      wgt[(size_t)t * ldk + top + lane] = gt;
+    }
   }
 }
 
@@ -667,17 +673,17 @@ GF_EXPORT int gf_moe_route(const float* logits, int T, int E, int top, int renor
 // See moe_route_grouped_kernel.
 GF_EXPORT int gf_moe_route_grouped(const float* logits, int ld, int T, int E, int identity, int top,
                                    int groups, int keep, const float* correction, int gate_col,
-                                   int* idx, float* wgt, float* identity_w, float* gate,
+                                   int always, int* idx, float* wgt, float* identity_w, float* gate,
                                    void* stream) {
   if (T <= 0) return 0;
   if (E <= 0 || E > kMaxExperts || identity < 0 || identity > E || top < 1 || groups < 1 ||
       E % groups || keep < 1 || keep > groups || top > E / groups * keep || ld < E ||
-      (gate && (gate_col < 0 || gate_col >= ld)))
+      gate_col >= ld || ((gate || always) && gate_col < 0) || always < 0 || always > 32)
     return -3;
 #define GF_GO(SLOTS)                                                                              \
   return launch_kernel(moe_route_grouped_kernel<SLOTS>, dim3((T + 3) / 4), dim3(128), 0,          \
                        (cudaStream_t)stream, logits, ld, T, E, identity, top, groups, keep,       \
-                       correction, gate_col, idx, wgt, identity_w, gate)
+                       correction, gate_col, always, idx, wgt, identity_w, gate)
   if (E <= 32) GF_GO(1);
   if (E <= 64) GF_GO(2);
   GF_GO(kRouteSlots);

@@ -32,7 +32,7 @@ TCGEN05_MIN_PAIRS = 1024
 # Up to this many pairs (decode steps of few requests) the products run on the kernel that streams
 # an expert's rows once for up to eight pairs; it keeps the rows in shared memory, which bounds the
 # reduction size.
-FEW_MAX_PAIRS = 16
+FEW_MAX_PAIRS = 20
 FEW_MAX_K = 4096
 
 
@@ -77,7 +77,7 @@ def route(logits: torch.Tensor, top: int, renormalize: bool, score: str = "softm
 
 
 def route_grouped(logits: torch.Tensor, experts: int, identity: int, top: int, correction=None,
-                  groups: int = 1, keep: int = 1, gate_col: int | None = None):
+                  groups: int = 1, keep: int = 1, gate_col: int | None = None, always: int = 0):
     """fp32 rows ``[T, >= experts + identity]`` (``identity`` experts without matrices are the last of
     the router's outputs) -> ``(experts [T, top] int32, weights [T, top], identity weights [T] or
     None, gates [T] or None)``, fp32.  Scores: the softmax over all outputs.  Choice scores: with
@@ -85,7 +85,9 @@ def route_grouped(logits: torch.Tensor, experts: int, identity: int, top: int, c
     (equal, of neighbours) with the largest best choice score can be chosen; the ``top`` with the
     largest choice scores are, lowest index among equals; the weights are their scores.  A chosen
     identity expert is ``-1`` with weight 0, its score counts in the identity weight.  ``gate_col``:
-    the column whose sigmoid is the token's gate."""
+    the column whose sigmoid is the token's gate.  ``always``: every token also has that many experts
+    behind the routed ones (``experts``, ``experts + 1``, ...) with its gate as their weight; the results
+    then have ``top + always`` columns."""
     _cuda(logits, correction)
     assert logits.dtype == torch.float32 and logits.dim() == 2 and logits.is_contiguous()
     T, ld = logits.shape
@@ -93,14 +95,15 @@ def route_grouped(logits: torch.Tensor, experts: int, identity: int, top: int, c
     assert correction is None or (correction.dtype == torch.float32 and correction.numel() == E
                                   and correction.is_contiguous())
     dev = logits.device
-    idx = torch.empty((T, top), dtype=torch.int32, device=dev)
-    wgt = torch.empty((T, top), dtype=torch.float32, device=dev)
+    idx = torch.empty((T, top + always), dtype=torch.int32, device=dev)
+    wgt = torch.empty((T, top + always), dtype=torch.float32, device=dev)
     idw = torch.empty((T,), dtype=torch.float32, device=dev) if identity else None
-    gate = torch.empty((T,), dtype=torch.float32, device=dev) if gate_col is not None else None
+    gate = torch.empty((T,), dtype=torch.float32, device=dev) \
+        if gate_col is not None and not always else None
     f = _fn("moe", "gf_moe_route_grouped",
-            [c_void_p] + [c_int] * 7 + [c_void_p, c_int] + [c_void_p] * 5)
+            [c_void_p] + [c_int] * 7 + [c_void_p, c_int, c_int] + [c_void_p] * 5)
     rc = f(_p(logits), ld, T, E, int(identity), int(top), int(groups), int(keep), _p(correction),
-           int(gate_col or 0), _p(idx), _p(wgt), _p(idw), _p(gate), _stream())
+           -1 if gate_col is None else int(gate_col), int(always), _p(idx), _p(wgt), _p(idw), _p(gate), _stream())
     if rc == -3:
         raise ValueError(f"the router kernel takes up to {MAX_EXPERTS} outputs in equal groups and no "
                          f"more choices than the kept groups hold; got {E} outputs, {groups} groups, "

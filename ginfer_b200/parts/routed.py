@@ -130,6 +130,10 @@ class RoutedExperts(FeedForward):
 register_feed_forward("routed_experts", RoutedExperts)
 
 
+# A shared expert of up to this many times the experts' size runs as that many of them.
+MAX_ALWAYS = 8
+
+
 class GroupRoutedGLU(RoutedGLU):
     """A :class:`RoutedGLU` chosen in groups.  Router scores ``s``: softmax over ALL outputs, ``experts``
     of them with matrices and then ``identity`` experts without (their output is their input).  Choice
@@ -138,9 +142,11 @@ class GroupRoutedGLU(RoutedGLU):
     the largest choice scores are chosen; the weights are their ``s``.  ``shared_size`` > 0: a shared
     expert of the same form runs for every token, times ``sigmoid(<prefix>.shared.sg h)``.
 
-    The shared gate's logit is one more row of the router's product.  The output is left as a sum
-    (:class:`TermSum`): the chosen experts' rows, the input times the identity weights, and the shared
-    expert's output times its gate."""
+    The shared gate's logit is one more row of the router's product.  A shared expert whose size is a
+    multiple of the experts' is that many more experts which every token has, with its gate as weight (an
+    expert of ``n F`` channels is the sum of ``n`` experts of ``F``), so that it needs no products of its
+    own.  The output is left as a sum (:class:`TermSum`): the chosen experts' rows, the input times the
+    identity weights, and, if it runs by itself, the shared expert's output times its gate."""
 
     can_defer_sum = False
     defers_terms = True
@@ -154,6 +160,8 @@ class GroupRoutedGLU(RoutedGLU):
         self.top, self.identity = int(top_k), int(identity)
         self.groups, self.keep, self.shared_size = int(groups), int(keep_groups), int(shared_size)
         outputs = self.E + self.identity
+        n, rest = divmod(self.shared_size, self.intermediate_size)
+        self.always = n if not rest and n <= MAX_ALWAYS and self.E + n <= moe.MAX_EXPERTS else 0
         if outputs > moe.MAX_EXPERTS:
             raise ValueError(f"{outputs} router outputs are over the kernel's {moe.MAX_EXPERTS}")
         if self.groups < 1 or outputs % self.groups or not (1 <= self.keep <= self.groups):
@@ -180,7 +188,14 @@ class GroupRoutedGLU(RoutedGLU):
         self.router = ops.Linear(joined_rows(rows), None, out_dtype=torch.float32)
         self.correction = tensors[p + "correction"].float().contiguous()
         self.shared = self.shared_down = None
-        if self.shared_size:
+        if self.always:
+            f, h, n = self.intermediate_size, self.hidden_size, self.always
+            gu = torch.stack([tensors[p + "shared.gate"], tensors[p + "shared.up"]],
+                             dim=1).reshape(n, 2 * f, h)
+            down = tensors[p + "shared.down"].view(h, n, f).transpose(0, 1)
+            self.w_gate_up = torch.cat([self.w_gate_up, gu]).contiguous()
+            self.w_down = torch.cat([self.w_down, down]).contiguous()
+        elif self.shared_size:
             self.shared = ops.GatedLinear(tensors[p + "shared.gate"], tensors[p + "shared.up"],
                                           clamped=(self.limit, self.alpha, self.up_shift))
             self.shared_down = ops.Linear(tensors[p + "shared.down"], None, out_dtype=torch.float32)
@@ -189,9 +204,10 @@ class GroupRoutedGLU(RoutedGLU):
         T = x.shape[0]
         idx, wgt, idw, gate = moe.route_grouped(
             self.router(x), self.E, self.identity, self.top, self.correction, self.groups, self.keep,
-            self.E + self.identity if self.shared_size else None)
-        plan = moe.Plan(idx, self.E, moe.kernel_for(
-            x, T * self.top, (self.hidden_size, self.intermediate_size),
+            self.E + self.identity if self.shared_size else None, self.always)
+        top = self.top + self.always
+        plan = moe.Plan(idx, self.E + self.always, moe.kernel_for(
+            x, T * top, (self.hidden_size, self.intermediate_size),
             (self.intermediate_size, self.hidden_size)))
         y = moe.grouped_glu(x, self.w_gate_up, plan, self.limit, self.alpha, self.up_shift,
                             act=self.act)
@@ -201,7 +217,7 @@ class GroupRoutedGLU(RoutedGLU):
             terms.append((self.shared_down(self.shared(x)), 1.0, gate))
         if idw is not None:
             terms.append((x, 1.0, idw))
-        out = TermSum(terms, PairSum(rows, plan.pos_of_pair, wgt, self.top,
+        out = TermSum(terms, PairSum(rows, plan.pos_of_pair, wgt, top,
                                      lambda: moe.combine(rows, plan, wgt, T)))
         return out if defer_terms else out.materialize()
 

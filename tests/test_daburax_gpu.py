@@ -554,6 +554,10 @@ def test_routing_in_groups(E, identity, top, groups, keep):
             close(idw[t], sum([s[t, e] for e in want if e >= E], torch.zeros((), dtype=F64)), 1e-6)
     assert identity or idw is None
     close(gate, torch.sigmoid(z[:, n + 1].double()), 1e-6)
+    more, w2, _, none = moe.route_grouped(z.cuda(), E, identity, top, corr.cuda(), groups, keep, n + 1, 3)
+    assert none is None and torch.equal(more[:, :top], idx) and torch.equal(w2[:, :top], wgt)
+    assert more[:, top:].tolist() == [[E, E + 1, E + 2]] * T
+    assert torch.equal(w2[:, top:], gate[:, None].expand(-1, 3))
     with pytest.raises(ValueError):
         moe.route_grouped(z.cuda(), E, identity, n + 1, corr.cuda(), groups, keep)
 
@@ -565,18 +569,21 @@ def test_ties_go_to_the_lower_index():
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("SF", [80, 96, 48])
 @pytest.mark.parametrize("T", [1, 3, 40, 700])
-def test_routed_feed_forward_with_identities_and_a_shared_expert(T, dtype):
+def test_routed_feed_forward_with_identities_and_a_shared_expert(T, SF, dtype):
     """The whole part, its sum formed by itself (``materialize``), on every kind of grouped product (a
-    handful of pairs, tiles, the persistent kernel); also when every token chooses identities only."""
+    handful of pairs, tiles, the persistent kernel); also when every token chooses identities only; a
+    shared expert with products of its own and one that is as large as one or two experts."""
     from ginfer_b200.parts import PartSpec, make_part
     g = torch.Generator().manual_seed(T)
-    W, F, E, I, SF = 64, 48, 6, 2, 80
+    W, F, E, I = 64, 48, 6, 2
     part = make_part("feed_forward", PartSpec("group_routed_glu", dict(
         hidden_size=W, intermediate_size=F, num_experts=E, top_k=2, identity=I, groups=4, keep_groups=2,
         shared_size=SF)))
     t = {s.name: torch.randn(s.shape, generator=g) * (s.shape[-1] ** -0.5 if len(s.shape) == 2 else 0.2)
          for s in part.tensor_specs()}
+    assert part.always == (SF // F if SF % F == 0 else 0)
     t["mlp.router"] *= 6.0
     x = torch.randn(T, W, generator=g)
     for only_identity in (False, True):
